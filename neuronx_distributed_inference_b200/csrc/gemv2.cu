@@ -1,7 +1,7 @@
-// GEMV v2: TMA (3-D tensor map, UTMALDG) mbarrier-pipelined weight-streaming skinny GEMM for decode
+// GEMV v2: TMA (3-D tensor map) mbarrier-pipelined weight-streaming skinny GEMM for decode
 //          Y[T<=8, N] = f( rmsnorm(X)[T,K] · W[N,K]^T )      (+ fused one-shot all-reduce over NVLink)
 //
-// Design (round 2):
+// Design:
 //   * ONE elected producer thread streams W with TMA tensor loads (cp.async.bulk.tensor.3d, completion on an
 //     mbarrier): W[N,K] is described as a 3-D tensor {64 k, K/64 groups, N rows}; one instruction fetches the box
 //     {64, 2, 16} = 16 weight rows x 128 k = 4 KB into a 128B-swizzled stage.
