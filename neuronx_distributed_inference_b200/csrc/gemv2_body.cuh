@@ -50,7 +50,7 @@ __device__ __forceinline__ void tma_load_3d(void* smem_dst, const CUtensorMap* t
       : "memory");
 }
 // Explicit shared-space accesses by 32-bit shared address.  The staging areas are carved out of dynamic shared memory at run
-// time; through plain pointers the address space is lost and loads / stores are generic (LD.E / ST.E) for every
+// time; through plain pointers the address space is lost and loads / stores are generic for every
 // fragment — measured as a uniform 1.5x slowdown of the streaming loop.
 __device__ __forceinline__ uint4 lds128(uint32_t a) {
   uint4 r;

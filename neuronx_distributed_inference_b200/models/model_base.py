@@ -182,6 +182,68 @@ class ConvPreNormDecoderLayer(nn.Module):
         return x, y
 
 
+class HyperConnectionDecoderLayer(nn.Module):
+    """Pre-norm block over ``S`` parallel fp32 residual streams.  Sublayer ``q`` (1: mixer, 2: feed-forward) reads one weighted sum of the
+    streams and its result is written back to all of them, while the streams are mixed with one another::
+
+        u = sum_s in_q[s] x_s;   y = sublayer(c(norm_q(u)));   x_t <- sum_s mix_q[s, t] x_s + out_q[t] y
+
+    ``norm_q`` is an RMS norm (weight over the width, or one number); the mixer's read also passes ``c(h) = h + conv(h)``, a depthwise causal
+    convolution over ``taps`` positions of the normalised rows (0: none), whose last ``taps - 1`` rows are carried per sequence in a state
+    line (fp32, one per RUN of the block).  Write-back, mixing, the next sublayer's weighted sum, norm, convolution and the carried rows are
+    ONE kernel (``ops.stream_mix_norm_conv``), so the result of a block's last sublayer is handed on unwritten: ``forward`` takes and
+    returns ``(x, pending)``, ``pending = (y, mix, out)``; ``finish`` applies it.  ``x`` is ``[B, T, S, W]``, or ``[B, T, W]`` before the
+    first write-back (all streams equal)."""
+    mlp_is_moe = False
+
+    def __init__(self, mixer: nn.Module, mlp: Optional[nn.Module], norm1: nn.Module, norm2: Optional[nn.Module], width: int, streams: int,
+                 taps: int, layer_idx: int = 0, device=None):
+        super().__init__()
+        self.mixer, self.mlp, self.norm1, self.norm2, self.layer_idx = mixer, mlp, norm1, norm2, layer_idx
+        par = lambda *s: nn.Parameter(torch.zeros(*s, dtype=torch.float32, device=device), requires_grad=False)      # noqa: E731
+        self.conv1_weight = par(width, taps) if taps else None
+        self.in1, self.out1, self.mix1 = par(streams), par(streams), par(streams, streams)
+        if mlp is not None:
+            self.in2, self.out2, self.mix2 = par(streams), par(streams), par(streams, streams)
+
+    def _state(self, run) -> str:
+        return f"stream_mix_conv.run{run}"
+
+    def state_specs(self, run=0):
+        specs = dict(getattr(self.mixer, "state_specs", lambda run: {})(run))
+        w = self.conv1_weight
+        if w is not None and w.shape[1] > 1:
+            specs[self._state(run)] = ((w.shape[1] - 1, w.shape[0]), torch.float32)
+        return specs
+
+    @staticmethod
+    def finish(x, pending, in_w, norm_w=None, eps=1e-6, lp_dtype=None, conv=None, state=None, meta=None):
+        """Write a handed-on result back to the streams and read them with the weights ``in_w`` (then norm, convolution)."""
+        y, mix, out = pending or (None, None, None)
+        ex = meta.extras if meta is not None else {}
+        return ops.stream_mix_norm_conv(x, y, mix, out, in_w, norm_w, conv, state, ex.get("state_lines"), ex.get("ctx_len"), ex.get("q_len"), eps,
+                                        lp_dtype)
+
+    def forward(self, x, pending, meta, kv_mgr, cache_index=None):
+        run = self.layer_idx if cache_index is None else cache_index
+        dtype, conv = meta.extras["act_dtype"], self.conv1_weight
+        state = kv_mgr.states.tensor(self._state(run)) if conv is not None and conv.shape[1] > 1 else None
+        x, h = self.finish(x, pending, self.in1, self.norm1.weight, self.norm1.variance_epsilon, dtype, conv, state, meta)
+        pending = (self.mixer(h, meta, kv_mgr, cache_index=run), self.mix1, self.out1)
+        if self.mlp is not None:
+            x, h = self.finish(x, pending, self.in2, self.norm2.weight, self.norm2.variance_epsilon, dtype, meta=meta)
+            router = getattr(self.mlp, "router", None)
+            if getattr(router, "by_token", False):
+                key = ("route", self.layer_idx)
+                if key not in meta.extras:
+                    meta.extras[key] = router(meta.extras["token_ids"], meta.extras["q_len"])[1:]
+                y = self.mlp(h, route=meta.extras[key])
+            else:
+                y = self.mlp(h)
+            pending = (y, self.mix2, self.out2)
+        return x, pending
+
+
 class SandwichNormDecoderLayer(nn.Module):
     """Block on an fp32 residual stream whose sublayers are normalised on BOTH sides, with a residual multiplier and a layer scale:
     ``r = mixer(norm1(x))``, ``x += mult * ls1 * norm1b(r)``, then, when the block has an MLP, ``r = mlp(norm2(x))``, ``x += mult * ls2 * norm2b(r)``.

@@ -58,6 +58,17 @@ def load_state_dict(path: str) -> Dict[str, torch.Tensor]:
     raise FileNotFoundError(f"no checkpoint files found under {path}")
 
 
+def tensor_shapes(path: str) -> Dict[str, tuple]:
+    """Shapes of a checkpoint folder's tensors from the safetensors headers alone (no data is read)."""
+    from safetensors import safe_open
+    shapes = {}
+    for f in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+        with safe_open(f, framework="pt") as h:
+            for k in h.keys():
+                shapes[k] = tuple(h.get_slice(k).get_shape())
+    return shapes
+
+
 def save_state_dict_safetensors(state_dict: Dict[str, torch.Tensor], out_dir: str, max_shard_size: int = 5 << 30):
     """Write (sharded) safetensors + index, HF-compatible."""
     from safetensors.torch import save_file

@@ -68,11 +68,27 @@ class RouterTopK(nn.Module):
         return logits, w, idx
 
 
+class TableRouter(nn.Module):
+    """No scores: row ``token id`` of an integer table ``[vocab, top_k]`` lists the experts of a token, each with weight ``1 / top_k``.
+    The routing of a token is the same wherever it stands, so a block that runs several times per forward routes once."""
+    by_token = True
+
+    def __init__(self, num_experts: int, top_k: int, vocab_size: int, device=None):
+        super().__init__()
+        self.num_experts, self.top_k = num_experts, top_k
+        self.table = nn.Parameter(torch.zeros(vocab_size, top_k, dtype=torch.int32, device=device), requires_grad=False)
+
+    def forward(self, token_ids: torch.Tensor, q_len: torch.Tensor):
+        w, idx = ops.table_route(self.table, token_ids, q_len)
+        return None, w, idx
+
+
 class ExpertMLPs(nn.Module):
     def __init__(self, num_experts: int, hidden_size: int, intermediate_size: int, hidden_act: str = "silu",
                  dtype=torch.float32, bias: bool = False, device=None, ep_group: Optional[Group] = None,
-                 moe_tp_group: Optional[Group] = None, act_fn: Optional[Callable] = None, gated: bool = True):
-        """``gated=False``: plain two-matrix experts ``down(act(up(x)))`` (Nemotron-H / Nemotron-3: squared ReLU); ``gate_up_proj`` is then
+                 moe_tp_group: Optional[Group] = None, act_fn: Optional[Callable] = None, gated: bool = True, act_params=None):
+        """``hidden_act="clamped_glu"``: the clamped, shifted gate product of :class:`ClampedGLUMLP` with ``act_params = (limit, alpha)``.
+        ``gated=False``: plain two-matrix experts ``down(act(up(x)))`` (Nemotron-H / Nemotron-3: squared ReLU); ``gate_up_proj`` is then
         just the up projection ``[E, I, H]``."""
         super().__init__()
         self.gated = gated
@@ -84,10 +100,12 @@ class ExpertMLPs(nn.Module):
         self.I_local = intermediate_size // tp
         self.expert_offset = self.ep_group.rank * self.E_local
         if gated:
-            self.act = {"silu": "silu_mul", "swish": "silu_mul", "gelu": "gelu_mul", "gelu_pytorch_tanh": "gelu_tanh_mul"}[hidden_act]
+            self.act = {"silu": "silu_mul", "swish": "silu_mul", "gelu": "gelu_mul", "gelu_pytorch_tanh": "gelu_tanh_mul",
+                        "clamped_glu": "clamped_glu"}[hidden_act]
         else:
             self.act = {"swish": "silu", "gelu_pytorch_tanh": "gelu_tanh"}.get(hidden_act, hidden_act)
         self.act_fn = act_fn
+        self.act_params = act_params
         nproj = 2 if gated else 1
         self.gate_up_proj = nn.Parameter(torch.empty(self.E_local, nproj * self.I_local, hidden_size, dtype=dtype, device=device),
                                          requires_grad=False)
@@ -123,7 +141,8 @@ class ExpertMLPs(nn.Module):
 
     def forward(self, x2: torch.Tensor, topk_w: torch.Tensor, topk_i: torch.Tensor, scale_input: bool = False) -> torch.Tensor:
         return ops.moe_experts(x2, self.gate_up_proj, self.down_proj, topk_w, topk_i, self.act, self.expert_offset,
-                               self.gate_up_bias, self.down_bias, self.act_fn, scale_input, self.gate_up_scale, self.down_scale)
+                               self.gate_up_bias, self.down_bias, self.act_fn, scale_input, self.gate_up_scale, self.down_scale,
+                               act_params=self.act_params)
 
 
 class MoE(nn.Module):
@@ -148,11 +167,12 @@ class MoE(nn.Module):
         self.last_router_logits = None
         self.last_expert_index = None
 
-    def forward(self, x, norm_weight=None, norm_eps=1e-6, norm_offset=0.0, residual=None, padding_mask=None):
+    def forward(self, x, norm_weight=None, norm_eps=1e-6, norm_offset=0.0, residual=None, padding_mask=None, route=None):
+        """``route``: (weights, expert ids) decided beforehand (:class:`TableRouter`) instead of by ``router(x)``."""
         shape = x.shape
         xn = ops.rmsnorm(x, norm_weight, norm_eps, norm_offset) if norm_weight is not None else x
         x2 = xn.reshape(-1, shape[-1])
-        logits, w, idx = self.router(x2)
+        logits, w, idx = self.router(x2) if route is None else (None, *route)
         if self.return_router_logits:
             self.last_router_logits = logits
         if self.return_expert_index:

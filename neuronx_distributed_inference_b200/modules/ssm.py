@@ -1,4 +1,5 @@
-"""Recurrent mixers on ragged rows with carried state (chunked prompts, mixed prefill / decode batches): Mamba-2 and the gated delta rule.
+"""Recurrent mixers on ragged rows with carried state (chunked prompts, mixed prefill / decode batches): Mamba-2, the gated delta rule (one
+decay per head, or one per head and key channel) and linear attention with a fixed decay per head.
 
 ``in_proj`` rows are ``[z: inner | x: inner | B: G N | C: G N | dt: heads]``.  x, B and C pass a depthwise causal convolution (+bias)
 and SiLU; ``dt = softplus(dt + dt_bias)``; per head ``S <- exp(-exp(A_log) dt) S + dt B x^T`` (fp32, ``[N, head_dim]``),
@@ -118,3 +119,100 @@ class RaggedGatedDeltaMixer(nn.Module):
         ops.short_conv_update(u, cst, lines, ctx, qlen)
         o = ops.gated_delta_scan(qkv, beta, a, self.A_log, self.dt_bias, sst, lines, ctx, qlen, H, self.n_qk, self.D, self.Dv, self.UNIT_EPS)
         return self.out_proj(ops.head_rmsnorm_gate(o, self.norm_weight, H, self.eps, gate, "silu", out_dtype=p.dtype))
+
+
+class RaggedChannelDeltaMixer(nn.Module):
+    """Gated delta rule whose state decays per head AND KEY CHANNEL, with low-rank decay and gate projections.  Projection rows are
+    ``[q: n_qk D | k: n_qk D | v: heads Dv | b: heads | a: decay_rank | g: gate_rank]`` in one GEMM; a second GEMM over the last two slices
+    with the block-diagonal weight ``[[W_a2, 0], [0, W_g2]]`` gives the raw decays (heads D) and the gate (heads Dv).  What differs from
+    :class:`RaggedGatedDeltaMixer`: ``decay = exp(-exp(A_log_h) * softplus(a + dt_bias))`` has one value per head and key channel, every row
+    of the state shrinks by its own, and the gate is a sigmoid.  The state ``[heads, Dv, D]`` keeps the key channels of a value channel
+    together.  ``run`` (``cache_index``): a block that runs several times per forward has a state line set per run.  CUDA
+    (csrc/linear_scan.cu): delta_front, channel_delta_scan; csrc/seqmix.cu: head_rmsnorm_gate."""
+    UNIT_EPS = 1e-6      # inside the root of the q / k unit norms (fixed by the rule)
+
+    def __init__(self, hidden_size: int, num_heads: int, num_qk_heads: int, head_dim: int, v_head_dim: int, decay_rank: int, gate_rank: int,
+                 conv_taps: int, eps: float, layer_idx: int, dtype=torch.bfloat16, device=None, tp_group=None):
+        super().__init__()
+        if num_heads % num_qk_heads:
+            raise ValueError("gated delta rule: value heads must be a multiple of q / k heads")
+        if tp_group is not None and tp_group.size != 1:
+            raise NotImplementedError("ragged channel-delta mixer: tensor parallel degree 1")
+        self.nh, self.n_qk, self.D, self.Dv = num_heads, num_qk_heads, head_dim, v_head_dim
+        self.taps, self.eps, self.layer_idx, self.ranks = conv_taps, eps, layer_idx, decay_rank + gate_rank
+        self.inner = num_heads * v_head_dim
+        self.conv_dim = 2 * num_qk_heads * head_dim + self.inner
+        col = lambda i, o: ColumnParallelLinear(i, o, bias=False, gather_output=False, dtype=dtype, device=device, tensor_model_parallel_group=tp_group)      # noqa: E731
+        self.in_proj = col(hidden_size, self.conv_dim + num_heads + self.ranks)
+        self.low_rank_up = col(self.ranks, num_heads * head_dim + self.inner)
+        self.out_proj = RowParallelLinear(self.inner, hidden_size, bias=False, input_is_parallel=True, dtype=dtype, device=device,
+                                          tensor_model_parallel_group=tp_group)
+        f32 = dict(dtype=torch.float32, device=device)
+        self.conv_weight = nn.Parameter(torch.zeros(self.conv_dim, conv_taps, **f32), requires_grad=False)
+        self.dt_bias = nn.Parameter(torch.zeros(num_heads * head_dim, **f32), requires_grad=False)
+        self.A_log = nn.Parameter(torch.zeros(num_heads, **f32), requires_grad=False)
+        self.norm_weight = nn.Parameter(torch.ones(v_head_dim, **f32), requires_grad=False)
+
+    @staticmethod
+    def block_diagonal(a, g):
+        """``[[a, 0], [0, g]]``: the two second projections as one matrix over the stacked low-rank rows."""
+        return torch.block_diag(a, g)
+
+    def _names(self, run):
+        run = self.layer_idx if run is None else run
+        return f"channel_delta_conv.run{run}", f"channel_delta_state.run{run}"
+
+    def state_specs(self, cache_index=None):
+        conv, state = self._names(cache_index)
+        return {conv: (self.taps - 1, self.conv_dim), state: ((self.nh, self.Dv, self.D), torch.float32)}
+
+    def forward(self, x, meta, kv_mgr, cache_index=None):
+        ex = meta.extras
+        where = (ex["state_lines"], ex["ctx_len"], ex["q_len"])
+        p = self.in_proj(x)
+        Cd, H = self.conv_dim, self.nh
+        up = self.low_rank_up(p[..., Cd + H:Cd + H + self.ranks].contiguous())
+        a, gate = up[..., :H * self.D], up[..., H * self.D:]
+        conv, state = (kv_mgr.states.tensor(n) for n in self._names(cache_index))
+        qkv, decay, beta = ops.delta_front(p, p[..., Cd:Cd + H], a, self.conv_weight, self.A_log, self.dt_bias, conv, *where, H, self.n_qk,
+                                           self.D, self.Dv, self.UNIT_EPS)
+        o = ops.channel_delta_scan(qkv, decay, beta, state, *where, H, self.n_qk, self.D, self.Dv)
+        return self.out_proj(ops.head_rmsnorm_gate(o, self.norm_weight, H, self.eps, gate, "sigmoid", out_dtype=p.dtype))
+
+
+class RaggedDecayMixer(nn.Module):
+    """Linear attention with a fixed decay per head on ragged rows.  Projection rows are ``[q: heads D | k: heads D | v: heads Dv | gate:
+    heads Dv]`` in one GEMM; q, k and v pass SiLU; per head the fp32 state (``[Dv, D]``) does ``M <- decay M + outer(k, v)``, ``y = M' q``.
+    The heads' outputs are RMS-normalised together (weight over all channels), multiplied by ``sigmoid(gate)`` and projected out.  ``decays``
+    are constants of the design, one per head.  CUDA: csrc/linear_scan.cu (decay_scan: recurrent form, and a chunked form on tensor cores
+    for bf16 portions), csrc/seqmix.cu (group_rmsnorm with a gate)."""
+
+    def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, decays, eps: float, layer_idx: int,
+                 dtype=torch.bfloat16, device=None, tp_group=None):
+        super().__init__()
+        if len(decays) != num_heads:
+            raise ValueError("one decay per head")
+        if tp_group is not None and tp_group.size != 1:
+            raise NotImplementedError("ragged decay mixer: tensor parallel degree 1")
+        self.nh, self.D, self.Dv, self.eps, self.layer_idx = num_heads, head_dim, v_head_dim, eps, layer_idx
+        self.inner, self.qkv = num_heads * v_head_dim, num_heads * (2 * head_dim + v_head_dim)
+        self.in_proj = ColumnParallelLinear(hidden_size, self.qkv + self.inner, bias=False, gather_output=False, dtype=dtype, device=device,
+                                            tensor_model_parallel_group=tp_group)
+        self.out_proj = RowParallelLinear(self.inner, hidden_size, bias=False, input_is_parallel=True, dtype=dtype, device=device,
+                                          tensor_model_parallel_group=tp_group)
+        self.register_buffer("decay", torch.tensor([float(d) for d in decays], dtype=torch.float32, device=device), persistent=False)
+        self.norm_weight = nn.Parameter(torch.ones(self.inner, dtype=torch.float32, device=device), requires_grad=False)
+
+    def _name(self, run):
+        return f"decay_state.run{self.layer_idx if run is None else run}"
+
+    def state_specs(self, cache_index=None):
+        return {self._name(cache_index): ((self.nh, self.Dv, self.D), torch.float32)}
+
+    def forward(self, x, meta, kv_mgr, cache_index=None):
+        ex = meta.extras
+        p = self.in_proj(x)
+        y = ops.decay_scan(p, self.decay, kv_mgr.states.tensor(self._name(cache_index)), ex["state_lines"], ex["ctx_len"], ex["q_len"], self.nh,
+                           self.D, self.Dv, True)
+        y = ops.group_rmsnorm(y, self.norm_weight, 1, self.eps, out_dtype=p.dtype, gate=p[..., self.qkv:], act="sigmoid")
+        return self.out_proj(y)

@@ -128,7 +128,14 @@ def linear(x, w, bias=None, norm_weight=None, norm_eps: float = 1e-6, norm_offse
                 y = _C().gemm(x2.contiguous(), w, bias, _ACT_CODES[act], r2, o2)
                 y = out if out is not None else y.view(*x.shape[:-1], y.shape[-1])
                 return y if (residual is None or r2 is not None) else y + residual
-    y = ref.linear(x, w, bias, norm_weight, norm_eps, norm_offset, act, scale)
+    if act == "silu_mul" and _mix_cuda(x) and w.dtype == x.dtype and scale is None and x.dim() >= 2:
+        # fp32 rows and sizes the GEMM kernels do not take: library product, then the gate product as one elementwise kernel
+        gu = ref.linear(x, w, bias, norm_weight, norm_eps, norm_offset)
+        g2 = gu.reshape(-1, gu.shape[-1])
+        n = g2.shape[-1] // 2
+        y = gated_act_mul(g2[:, :n], g2[:, n:], "silu").view(*gu.shape[:-1], n)
+    else:
+        y = ref.linear(x, w, bias, norm_weight, norm_eps, norm_offset, act, scale)
     y = y if residual is None else y + residual
     if out is not None:
         out.copy_(y)
@@ -379,8 +386,10 @@ def identity_expert_add(y, x, topk_w, topk_i, num_experts: int):
 
 
 def moe_experts(x, w_gate_up, w_down, topk_w, topk_i, act="silu_mul", expert_offset=0,
-                gate_up_bias=None, down_bias=None, act_fn=None, scale_input=False, gate_up_scale=None, down_scale=None):
+                gate_up_bias=None, down_bias=None, act_fn=None, scale_input=False, gate_up_scale=None, down_scale=None, act_params=None):
+    """``act_params``: constants of the activation (``"clamped_glu"``: limit, alpha)."""
     N = x.shape[0]
+    limit, alpha = (float(v) for v in act_params) if act == "clamped_glu" else (7.0, 1.702)
     if (act in _MOE_PLAIN_ACTS and _mix_cuda(x) and act_fn is None and gate_up_scale is None and down_scale is None and gate_up_bias is None
             and down_bias is None and not scale_input and w_gate_up.dtype == x.dtype and w_down.dtype == x.dtype and topk_i.dim() == 2
             and topk_i.shape[1] <= 64 and w_gate_up.shape[0] <= 512 and w_gate_up.is_contiguous() and w_down.is_contiguous()):
@@ -389,16 +398,16 @@ def moe_experts(x, w_gate_up, w_down, topk_w, topk_i, act="silu_mul", expert_off
         stats["moe_plain"] += 1
         tc = _MOE_GROUPED and x.dtype == torch.bfloat16 and x.shape[1] % 64 == 0 and w_down.shape[2] % 64 == 0 and N > GEMV_MAX_TOKENS
         return _C().moe_plain(x.contiguous(), w_gate_up, w_down, topk_w.float().contiguous(), topk_i.to(torch.int32).contiguous(),
-                              int(expert_offset), _MOE_PLAIN_ACTS[act], bool(tc), False)
+                              int(expert_offset), _MOE_PLAIN_ACTS[act], bool(tc), False, limit, alpha)
     bf16_shapes = x.dtype == torch.bfloat16 and x.shape[1] % 64 == 0 and w_down.shape[2] % 64 == 0
-    if (act == "silu_mul" and _mix_cuda(x) and not bf16_shapes and act_fn is None and gate_up_scale is None and down_scale is None
+    if (act in ("silu_mul", "clamped_glu") and _mix_cuda(x) and not bf16_shapes and act_fn is None and gate_up_scale is None and down_scale is None
             and gate_up_bias is None and down_bias is None and not scale_input and w_gate_up.dtype == x.dtype and w_down.dtype == x.dtype
             and topk_i.dim() == 2 and topk_i.shape[1] <= 64 and w_gate_up.shape[0] <= 512 and w_gate_up.is_contiguous() and w_down.is_contiguous()):
         # gated experts in fp32 or with sizes the tensor-core kernels do not take: the same permutation around the CUDA-core grouped
         # GEMMs, the gate product as an elementwise pass between them
         stats["moe_plain_gated"] += 1
         return _C().moe_plain(x.contiguous(), w_gate_up, w_down, topk_w.float().contiguous(), topk_i.to(torch.int32).contiguous(),
-                              int(expert_offset), _UNARY_ACTS["silu"], False, True)
+                              int(expert_offset), _CLAMPED_GLU if act == "clamped_glu" else _UNARY_ACTS["silu"], False, True, limit, alpha)
     if gate_up_scale is not None or down_scale is not None:
         # fp8 experts with dynamic activation quantisation asked for: W8A8 grouped GEMMs on the kind::f8f6f4 tensor-core path
         if (_use_cuda(x) and _MOE_GROUPED and _ACT_QUANT and N > GEMV_MAX_TOKENS and x.dtype == torch.bfloat16 and act in _MOE_ACTS
@@ -412,19 +421,19 @@ def moe_experts(x, w_gate_up, w_down, topk_w, topk_i, act="silu_mul", expert_off
                                     topk_i.to(torch.int32).contiguous(), int(expert_offset), _MOE_ACTS[act], bool(scale_input),
                                     None if gate_up_bias is None else gate_up_bias.contiguous(),
                                     None if down_bias is None else down_bias.contiguous(),
-                                    gate_up_scale.float().contiguous(), down_scale.float().contiguous())
+                                    gate_up_scale.float().contiguous(), down_scale.float().contiguous(), limit, alpha)
         # weight-only 8-bit experts: dequantise the selected experts on the fly
         return ref.moe_experts(x, w_gate_up, w_down, topk_w, topk_i, act, expert_offset, gate_up_bias, down_bias, act_fn, scale_input,
                                gate_up_scale, down_scale)
     # activations with a kernel implementation: the named GLU ones, or a callable that names its kernel twin (``kernel_act``)
     kact = act if act_fn is None else getattr(act_fn, "kernel_act", None)
-    if (_use_cuda(x) and x.dtype in _FAST_DTYPES and w_gate_up.dtype == x.dtype and act == "silu_mul"
+    if (_use_cuda(x) and x.dtype in _FAST_DTYPES and w_gate_up.dtype == x.dtype and act in ("silu_mul", "clamped_glu")
             and act_fn is None and gate_up_bias is None and down_bias is None and N <= GEMV_MAX_TOKENS and not scale_input
             and w_gate_up.is_contiguous() and w_down.is_contiguous() and topk_i.dim() == 2
             and x.shape[1] % 8 == 0 and w_down.shape[2] % 8 == 0 and max(x.shape[1], w_down.shape[2]) * 2 <= 65536):
         stats["moe_decode"] += 1
         return _C().moe_decode(x.contiguous(), w_gate_up, w_down, topk_w.float().contiguous(),
-                               topk_i.to(torch.int32).contiguous(), int(expert_offset))
+                               topk_i.to(torch.int32).contiguous(), int(expert_offset), _MOE_ACTS[act], limit, alpha)
     # prefill-sized batches: device-side permutation + grouped tcgen05 GEMMs (static shapes: replays under CUDA graphs)
     if (_use_cuda(x) and _MOE_GROUPED and x.dtype == torch.bfloat16 and w_gate_up.dtype == x.dtype and w_down.dtype == x.dtype
             and kact in _MOE_ACTS and topk_i.dim() == 2 and topk_i.shape[1] <= 64
@@ -435,15 +444,16 @@ def moe_experts(x, w_gate_up, w_down, topk_w, topk_i, act="silu_mul", expert_off
         return _C().moe_grouped(x.contiguous(), w_gate_up, w_down, topk_w.float().contiguous(), topk_i.to(torch.int32).contiguous(),
                                 int(expert_offset), _MOE_ACTS[kact], bool(scale_input),
                                 None if gate_up_bias is None else gate_up_bias.contiguous(),
-                                None if down_bias is None else down_bias.contiguous(), None, None)
+                                None if down_bias is None else down_bias.contiguous(), None, None, limit, alpha)
     return ref.moe_experts(x, w_gate_up, w_down, topk_w, topk_i, act, expert_offset, gate_up_bias, down_bias,
-                           act_fn, scale_input)
+                           act_fn, scale_input, act_params=act_params)
 
 
 _MOE_GROUPED = os.environ.get("NXDI_B200_MOE_GROUPED", "1") == "1"
-_MOE_ACTS = {"silu_mul": 1, "gelu_tanh_mul": 2, "gelu_mul": 3, "gpt_oss_glu": 4}
+_MOE_ACTS = {"silu_mul": 1, "gelu_tanh_mul": 2, "gelu_mul": 3, "gpt_oss_glu": 4, "clamped_glu": 4}      # 4 takes (limit, alpha); gpt_oss_glu: 7, 1.702
 _UNARY_ACTS = {"relu": 1, "relu2": 2, "silu": 3, "gelu_tanh": 4, "sigmoid": 5, "gelu": 6}         # codes of csrc/seqmix.cu (unary_act, moe_plain, gated_act_mul)
 _MOE_PLAIN_ACTS = _UNARY_ACTS
+_CLAMPED_GLU = 7         # moe_plain's code of the clamped gate product (gated experts only)
 
 
 def rmsnorm_quant(x, weight, eps, clamp=float("inf"), offset: float = 0.0):
@@ -548,13 +558,15 @@ def ssd_scan(xBC, dt_raw, z, A_log, dt_bias, D_skip, state, slots, ctx_len, q_le
     return ref.ssd_scan(xBC, dt_raw, z, A_log, dt_bias, D_skip, state, slots, ctx_len, q_len, n_heads, head_dim, n_state, n_groups)
 
 
-def group_rmsnorm(y, weight, groups: int, eps: float, out_dtype=None):
+def group_rmsnorm(y, weight, groups: int, eps: float, out_dtype=None, gate=None, act: str = "sigmoid"):
     od = out_dtype or y.dtype
-    if _use_cuda(y) and y.dtype == torch.float32 and od in _MIX_DTYPES:
+    if (_use_cuda(y) and y.dtype == torch.float32 and od in _MIX_DTYPES and (gate is None or (gate.dtype in _MIX_DTYPES and gate.stride(-1) == 1
+                                                                                          and gate.shape == y.shape and act in _UNARY_ACTS))):
         stats["group_rmsnorm"] += 1
         W = y.shape[-1]
-        return _C().group_rmsnorm(y.reshape(-1, W).contiguous(), weight, int(groups), float(eps), od == torch.bfloat16).view(y.shape)
-    return ref.group_rmsnorm(y, weight, groups, eps, out_dtype)
+        g2 = None if gate is None else gate if gate.dim() == 2 else gate.reshape(-1, W) if gate.is_contiguous() else _rows_view(gate)
+        return _C().group_rmsnorm(y.reshape(-1, W).contiguous(), weight, int(groups), float(eps), od == torch.bfloat16, g2, _UNARY_ACTS[act]).view(y.shape)
+    return ref.group_rmsnorm(y, weight, groups, eps, out_dtype, gate, act)
 
 
 def clamped_glu(gu, limit: float, alpha: float = 1.702):
@@ -639,12 +651,12 @@ def latent_prefill_on_tensor_cores(x, rank: int) -> bool:
 
 
 def gated_act_mul(gate, other, act: str = "gelu_tanh", act_on_other: bool = False):
-    if _mix_cuda(gate) and other.dtype == gate.dtype and other.stride(-1) == 1 and gate.is_contiguous() and act in _UNARY_ACTS \
-            and other.dim() == gate.dim() and other.shape == gate.shape:
+    if _mix_cuda(gate) and other.dtype == gate.dtype and other.stride(-1) == 1 and act in _UNARY_ACTS and other.shape == gate.shape \
+            and (gate.is_contiguous() or (gate.dim() == 2 and gate.stride(-1) == 1)):
         stats["gated_act_mul"] += 1
         C = gate.shape[-1]
         o2 = other if other.dim() == 2 else other.reshape(-1, C) if other.is_contiguous() else _rows_view(other)
-        return _C().gated_act_mul(gate.reshape(-1, C), o2, _UNARY_ACTS[act], bool(act_on_other)).view(gate.shape)
+        return _C().gated_act_mul(gate if gate.dim() == 2 else gate.reshape(-1, C), o2, _UNARY_ACTS[act], bool(act_on_other)).view(gate.shape)
     return ref.gated_act_mul(gate, other, act, act_on_other)
 
 
@@ -683,16 +695,16 @@ def stream_sandwich_norm(x, a=None, b=None, a_weight=None, b_weight=None, a_scal
 
 
 def head_norm_rope_append(p, n_q, n_kv, D, Dv, cos, sin, q_norm_w, k_norm_w, norm_at: int, eps: float, value_from_key: bool, k_cache, v_cache,
-                          block_table, ctx_len, q_len, out_dtype=None):
+                          block_table, ctx_len, q_len, out_dtype=None, n_v=None):
     """Per-head q / k RMS norm (before or after the rotation) + rotate-half rotation + paged cache write, ONE kernel (definition:
     ops/reference.py)."""
     if _mix_cuda(p) and p.stride(-1) == 1 and D <= 256 and k_cache.dtype == p.dtype and v_cache.dtype == p.dtype and (cos is None or cos.shape[-1] * 2 <= D):
         stats["head_norm_rope_append"] += 1
         f32 = lambda t: None if t is None else t.float().contiguous()          # noqa: E731
         return _C().head_norm_rope_append(p, int(n_q), int(n_kv), int(D), int(Dv), f32(cos), f32(sin), f32(q_norm_w), f32(k_norm_w), int(norm_at),
-                                          float(eps), bool(value_from_key), k_cache, v_cache, _i32(block_table), _i32(ctx_len), _i32(q_len))
+                                          float(eps), bool(value_from_key), k_cache, v_cache, _i32(block_table), _i32(ctx_len), _i32(q_len), int(n_kv if n_v is None else n_v))
     return ref.head_norm_rope_append(p, n_q, n_kv, D, Dv, cos, sin, q_norm_w, k_norm_w, norm_at, eps, value_from_key, k_cache, v_cache,
-                                     block_table, ctx_len, q_len, out_dtype)
+                                     block_table, ctx_len, q_len, out_dtype, n_v)
 
 
 def gated_delta_scan(qkv, beta_raw, a_raw, A_log, dt_bias, state, slots, ctx_len, q_len, n_heads, n_qk, D, Dv, unit_eps: float = 1e-6):
@@ -714,3 +726,64 @@ def head_rmsnorm_gate(y, weight, heads: int, eps: float, gate, act: str = "silu"
         return _C().head_rmsnorm_gate(y.reshape(-1, C).contiguous(), weight.float().contiguous(), int(heads), float(eps), g2, _UNARY_ACTS[act],
                                       od == torch.bfloat16).view(y.shape)
     return ref.head_rmsnorm_gate(y, weight, heads, eps, gate, act, out_dtype)
+
+
+# ---- several residual streams, differential attention, fixed and per-channel decays, routing by token id --------------------------------
+_MIX_MAX_STREAMS = 8
+
+
+def stream_mix_norm_conv(x, y, mix, out_w, in_w, norm_w, conv_w, state, slots, ctx_len, q_len, eps: float, lp_dtype=None):
+    """Update of several fp32 residual streams + the read, norm and short convolution of the next sublayer (+ the carried rows), ONE kernel
+    (definition: ops/reference.py)."""
+    S, W = in_w.shape[0], x.shape[-1]
+    taps = 1 if conv_w is None else conv_w.shape[1]
+    if (_use_cuda(x) and x.dtype == torch.float32 and (y is None or y.dtype in _MIX_DTYPES) and S <= _MIX_MAX_STREAMS and taps <= _MIX_MAX_TAPS
+            and W <= 16384 and (state is None or state.dtype == torch.float32)):
+        stats["stream_mix_norm_conv"] += 1
+        f32 = lambda t: None if t is None else t.float().contiguous()          # noqa: E731
+        i32 = lambda t: None if t is None else _i32(t)                         # noqa: E731
+        xn, r = _C().stream_mix_norm_conv(x.contiguous(), None if y is None else y.contiguous(), f32(mix), f32(out_w), f32(in_w), f32(norm_w),
+                                          f32(conv_w), state, i32(slots), i32(ctx_len), i32(q_len), float(eps), lp_dtype == torch.bfloat16)
+        return (x if y is None else xn), r
+    return ref.stream_mix_norm_conv(x, y, mix, out_w, in_w, norm_w, conv_w, state, slots, ctx_len, q_len, eps, lp_dtype)
+
+
+def paged_diff_attention(q, k_cache, v_cache, block_table, ctx_len, q_len, scale: float, lam, out_scale: float, eps: float, window: int = 0):
+    """Both maps of every head, their difference, its norm and scale in ONE kernel (definition: ops/reference.py)."""
+    if _mix_cuda(q) and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype and v_cache.shape[-1] <= _MIX_MAX_VDIM:
+        stats["paged_diff_attention"] += 1
+        return _C().paged_diff_attention(q.contiguous(), k_cache, v_cache, _i32(block_table), _i32(ctx_len), _i32(q_len), float(scale),
+                                         lam.float().contiguous(), float(out_scale), float(eps), int(window or 0))
+    return ref.paged_diff_attention(q, k_cache, v_cache, block_table, ctx_len, q_len, scale, lam, out_scale, eps, window)
+
+
+def delta_front(p, beta_raw, a_raw, conv_w, A_log, dt_bias, state, slots, ctx_len, q_len, n_heads: int, n_qk: int, D: int, Dv: int,
+                unit_eps: float = 1e-6):
+    if (_mix_cuda(p) and p.stride(-1) == 1 and beta_raw.dtype == p.dtype and a_raw.dtype == p.dtype and beta_raw.stride(-1) == 1
+            and a_raw.stride(-1) == 1 and conv_w.shape[1] <= _MIX_MAX_TAPS and D <= 256):
+        stats["delta_front"] += 1
+        return tuple(_C().delta_front(p, beta_raw, a_raw, conv_w, A_log, dt_bias, state, _i32(slots), _i32(ctx_len), _i32(q_len), int(n_heads),
+                                      int(n_qk), int(D), int(Dv), float(unit_eps)))
+    return ref.delta_front(p, beta_raw, a_raw, conv_w, A_log, dt_bias, state, slots, ctx_len, q_len, n_heads, n_qk, D, Dv, unit_eps)
+
+
+def channel_delta_scan(qkv, decay, beta, state, slots, ctx_len, q_len, n_heads: int, n_qk: int, D: int, Dv: int):
+    if _use_cuda(qkv) and qkv.dtype == torch.float32 and state.dtype == torch.float32 and D <= 256:
+        stats["channel_delta_scan"] += 1
+        return _C().channel_delta_scan(qkv.contiguous(), decay.contiguous(), beta.contiguous(), state, _i32(slots), _i32(ctx_len), _i32(q_len),
+                                       int(n_heads), int(n_qk), int(D), int(Dv))
+    return ref.channel_delta_scan(qkv, decay, beta, state, slots, ctx_len, q_len, n_heads, n_qk, D, Dv)
+
+
+def decay_scan(p, decay, state, slots, ctx_len, q_len, n_heads: int, D: int, Dv: int, silu: bool = True):
+    if _mix_cuda(p) and p.stride(-1) == 1 and state.dtype == torch.float32 and D <= 256:
+        stats["decay_scan"] += 1
+        return _C().decay_scan(p, decay, state, _i32(slots), _i32(ctx_len), _i32(q_len), int(n_heads), int(D), int(Dv), bool(silu))
+    return ref.decay_scan(p, decay, state, slots, ctx_len, q_len, n_heads, D, Dv, silu)
+
+
+def table_route(table, token_ids, q_len):
+    if _use_cuda(table) and table.dtype == torch.int32 and table.is_contiguous():
+        stats["table_route"] += 1
+        return tuple(_C().table_route(table, _i32(token_ids), _i32(q_len)))
+    return ref.table_route(table, token_ids, q_len)

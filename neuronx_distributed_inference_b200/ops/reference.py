@@ -310,11 +310,12 @@ def identity_expert_add(y, x, topk_w, topk_i, num_experts: int):
 
 
 def moe_experts(x, w_gate_up, w_down, topk_w, topk_i, act: str = "silu_mul", expert_offset: int = 0,
-                gate_up_bias=None, down_bias=None, act_fn=None, scale_input: bool = False, gate_up_scale=None, down_scale=None):
+                gate_up_bias=None, down_bias=None, act_fn=None, scale_input: bool = False, gate_up_scale=None, down_scale=None, act_params=None):
     """Dropless expert MLPs.  x [N,H]; w_gate_up [E_local, 2I, H] ([gate; up] rows, K-major like nn.Linear — the
     reference stores [E,H,2I]; K-major is what TMA/UMMA and the GEMV kernels stream); w_down
     [E_local, H, I]; experts owned here are [expert_offset, expert_offset+E_local).
-    -> partial output [N,H] (sum over owned experts; all-reduce across expert/tensor shards outside)."""
+    -> partial output [N,H] (sum over owned experts; all-reduce across expert/tensor shards outside).  ``act = "clamped_glu"``: the
+    product of :func:`clamped_glu` with ``act_params = (limit, alpha)``."""
     N, H = x.shape
     E = w_gate_up.shape[0]
     out = torch.zeros(N, H, dtype=torch.float32, device=x.device)
@@ -333,7 +334,7 @@ def moe_experts(x, w_gate_up, w_down, topk_w, topk_i, act: str = "silu_mul", exp
             h = (h.float() * gate_up_scale[e].float()).to(x.dtype)
         if gate_up_bias is not None:
             h = h + gate_up_bias[e].to(h.dtype)
-        h = act_fn(h) if act_fn is not None else activation(h, act)
+        h = act_fn(h) if act_fn is not None else clamped_glu(h, *act_params) if act == "clamped_glu" else activation(h, act)
         y = F.linear(h, w_down[e].to(x.dtype))
         if down_scale is not None:
             y = (y.float() * down_scale[e].float()).to(x.dtype)
@@ -559,11 +560,15 @@ def ssd_scan(xBC, dt_raw, z, A_log, dt_bias, D_skip, state, slots, ctx_len, q_le
     return y.reshape(B, T, inner) * F.silu(z.float())
 
 
-def group_rmsnorm(y, weight, groups: int, eps: float, out_dtype=None):
-    """RMS norm of ``groups`` equal parts of the last axis, each by its own root mean square, times ``weight``."""
+def group_rmsnorm(y, weight, groups: int, eps: float, out_dtype=None, gate=None, act: str = "sigmoid"):
+    """RMS norm of ``groups`` equal parts of the last axis, each by its own root mean square, times ``weight``; ``gate`` (the shape of
+    ``y``, possibly a strided slice of a wider row): times ``act(gate)`` after the norm."""
     yf = y.float().reshape(*y.shape[:-1], groups, y.shape[-1] // groups)
     yf = (yf * torch.rsqrt(yf.pow(2).mean(-1, keepdim=True) + eps)).reshape(y.shape)
-    return (yf * weight.float()).to(out_dtype or y.dtype)
+    yf = yf * weight.float()
+    if gate is not None:
+        yf = yf * activation(gate.float(), act)
+    return yf.to(out_dtype or y.dtype)
 
 
 def clamped_glu(gu, limit: float, alpha: float = 1.702):
@@ -727,18 +732,20 @@ def stream_sandwich_norm(x, a=None, b=None, a_weight=None, b_weight=None, a_scal
 
 
 def head_norm_rope_append(p, n_q: int, n_kv: int, D: int, Dv: int, cos, sin, q_norm_w, k_norm_w, norm_at: int, eps: float,
-                          value_from_key: bool, k_cache, v_cache, block_table, ctx_len, q_len, out_dtype=None):
+                          value_from_key: bool, k_cache, v_cache, block_table, ctx_len, q_len, out_dtype=None, n_v=None):
     """Front half of a grouped-query attention layer on ragged rows.  ``p`` [B, T, >= n_q D + n_kv D (+ n_kv Dv)] holds q | k | v
     (no v slice when ``value_from_key``: the raw k slice doubles as the value, untouched by norm or rotation, so ``Dv == D``).
     Every q and k head is RMS-normalised over its ``D`` channels (``norm_at`` 1: before the rotation, 2: after it, 0: not at all;
     ``q_norm_w`` / ``k_norm_w`` [D] are shared by the heads, ``None`` = no weight) and its first ``2 * cos.shape[-1]`` channels are
     rotated in the rotate-half layout (channel ``i`` pairs with ``i + R / 2``); ``cos = None`` skips the rotation.  Keys and values go
-    to the paged caches ``[blocks, page, n_kv, D | Dv]`` at position ``ctx_len + t``.  Returns q [B, T, n_q, D]."""
+    to the paged caches ``[blocks, page, n_kv, D]`` / ``[blocks, page, n_v, Dv]`` at position ``ctx_len + t``; ``n_v`` (default
+    ``n_kv``): value heads, when several key heads share one value head.  Returns q [B, T, n_q, D]."""
     B, T = p.shape[:2]
     Cq, Ck = n_q * D, n_kv * D
+    n_v = n_kv if n_v is None else n_v
     q = p[..., :Cq].float().reshape(B, T, n_q, D)
     k_raw = p[..., Cq:Cq + Ck].float().reshape(B, T, n_kv, D)
-    v = k_raw if value_from_key else p[..., Cq + Ck:Cq + Ck + n_kv * Dv].float().reshape(B, T, n_kv, Dv)
+    v = k_raw if value_from_key else p[..., Cq + Ck:Cq + Ck + n_v * Dv].float().reshape(B, T, n_v, Dv)
 
     def prep(x, w):
         if norm_at == 1:
@@ -761,7 +768,7 @@ def head_norm_rope_append(p, n_q: int, n_kv: int, D: int, Dv: int, cos, sin, q_n
     blk = torch.gather(block_table.long(), 1, (pos // page).clamp(0, block_table.shape[1] - 1))
     slot = (blk * page + pos % page)[ok]
     k_cache.view(-1, n_kv, D)[slot] = k[ok].to(k_cache.dtype)
-    v_cache.view(-1, n_kv, Dv)[slot] = v[ok].to(v_cache.dtype)
+    v_cache.view(-1, n_v, Dv)[slot] = v[ok].to(v_cache.dtype)
     return q.to(out_dtype or p.dtype)
 
 
@@ -802,3 +809,126 @@ def head_rmsnorm_gate(y, weight, heads: int, eps: float, gate, act: str = "silu"
     Dv = y.shape[-1] // heads
     yf = _norm_rows(y.float().reshape(*y.shape[:-1], heads, Dv), False, eps) * weight.float()
     return (yf.reshape(y.shape) * activation(gate.float(), act)).to(out_dtype or y.dtype)
+
+
+# ---- several residual streams, differential attention, fixed and per-channel decays, routing by token id --------------------------------
+def stream_mix_norm_conv(x, y, mix, out_w, in_w, norm_w, conv_w, state, slots, ctx_len, q_len, eps: float, lp_dtype=None):
+    """One update of ``S`` parallel fp32 residual streams and what the next sublayer reads from them::
+
+        x'_t = sum_s mix[s, t] x_s + out_w[t] * y          (all streams from the old ones; ``y = None``: x' = x)
+        u    = sum_s in_w[s] x'_s
+        h    = rms_unit(u) * norm_w                        (``norm_w`` [W] or one number; ``None``: h = u)
+        r_p  = h_p + sum_j conv_w[:, j] * h_(p - taps + 1 + j)            (over positions p; ``conv_w = None``: r = h)
+
+    ``x`` is ``[B, T, S, W]``, or ``[B, T, W]`` when all ``S = len(in_w)`` streams are still equal.  ``state`` [lines, taps - 1, W] fp32
+    holds the last ``taps - 1`` rows ``h`` of every sequence (line ``slots[b]``, zero when ``ctx_len`` is 0) and is ADVANCED by
+    ``q_len`` rows.  Everything is fp32.  Returns ``(x' [B, T, S, W], or x itself without y; r in lp_dtype, fp32 when None)``."""
+    S = in_w.shape[0]
+    xf = x.float()
+    xs = xf.unsqueeze(2).expand(-1, -1, S, -1) if xf.dim() == 3 else xf
+    if y is not None:
+        xs = torch.einsum("btsw,sd->btdw", xs, mix.float()) + out_w.float().view(1, 1, S, 1) * y.float().unsqueeze(2)
+    h = (xs * in_w.float().view(1, 1, S, 1)).sum(2)
+    if norm_w is not None:
+        h = h * torch.rsqrt(h.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()
+    r = h
+    if conv_w is not None:
+        if conv_w.shape[1] == 1:
+            r = h + h * conv_w[:, 0].float()
+        else:
+            r = h + short_conv(h, conv_w, None, state, slots, ctx_len, q_len)
+            short_conv_update(h, state, slots, ctx_len, q_len)
+    return (x if y is None else xs), (r if lp_dtype in (None, torch.float32) else r.to(lp_dtype))
+
+
+def paged_diff_attention(q, k_cache, v_cache, block_table, ctx_len, q_len, scale: float, lam, out_scale: float, eps: float, window: int = 0):
+    """Differential attention over the paged cache: every head has two maps, each a softmax attention of its own over the same values;
+    with their outputs ``a1`` and ``a2``, ``o = a1 - lam * a2`` is divided by its root mean square over the value channels (``eps``
+    under the root) and multiplied by ``out_scale``.  ``q`` [B, T, 2 H, D] and ``k_cache`` [blocks, page, 2 G, D] are laid out head by
+    head as (map 1, map 2), ``v_cache`` [blocks, page, G, Dv]; ``lam`` [1] fp32; ``window`` as in :func:`paged_window_attention`.
+    Returns [B, T, H * Dv]."""
+    B, T, H2, D = q.shape
+    blocks, page, G2, _ = k_cache.shape
+    Dv = v_cache.shape[3]
+    one = lambda m: paged_window_attention(q[:, :, m::2].float(), k_cache[:, :, m::2].float(), v_cache.float(), block_table, ctx_len, q_len,      # noqa: E731
+                                           scale, 0.0, window, 0)
+    o = (one(0) - lam.float() * one(1)).view(B, T, H2 // 2, Dv)
+    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * out_scale
+    return o.reshape(B, T, -1).to(q.dtype)
+
+
+def delta_front(p, beta_raw, a_raw, conv_w, A_log, dt_bias, state, slots, ctx_len, q_len, n_heads: int, n_qk: int, D: int, Dv: int,
+                unit_eps: float = 1e-6):
+    """What a gated delta rule with one decay per head and KEY CHANNEL reads.  ``p`` [B, T, >= 2 n_qk D + n_heads Dv] holds q | k | v
+    projections: every channel passes a short causal convolution (carried rows in ``state``, ADVANCED here) and SiLU, q and k heads are
+    scaled to unit length (``unit_eps`` under the root), q also by ``D^-1/2``.  ``decay = exp(-exp(A_log) * softplus(a_raw + dt_bias))``
+    with ``a_raw`` [B, T, n_heads D], ``A_log`` [n_heads], ``dt_bias`` [n_heads D]; ``b = sigmoid(beta_raw)``.  Returns
+    ``(q | k | v, decay, b)`` in fp32."""
+    B, T = p.shape[:2]
+    Cq, C = n_qk * D, 2 * n_qk * D + n_heads * Dv
+    u = p[..., :C]
+    y = short_conv(u, conv_w, None, state, slots, ctx_len, q_len, silu=True)
+    short_conv_update(u, state, slots, ctx_len, q_len)
+    unit = lambda x: (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) + unit_eps))          # noqa: E731
+    q = unit(y[..., :Cq].reshape(B, T, n_qk, D)) * D ** -0.5
+    k = unit(y[..., Cq:2 * Cq].reshape(B, T, n_qk, D))
+    qkv = torch.cat([q.reshape(B, T, Cq), k.reshape(B, T, Cq), y[..., 2 * Cq:]], -1)
+    decay = torch.exp(-torch.exp(A_log.float()).repeat_interleave(D) * F.softplus(a_raw.float() + dt_bias.float(), threshold=1e9))
+    return qkv, decay, torch.sigmoid(beta_raw.float())
+
+
+def channel_delta_scan(qkv, decay, beta, state, slots, ctx_len, q_len, n_heads: int, n_qk: int, D: int, Dv: int):
+    """Gated delta rule with one decay per head and key channel, on the rows :func:`delta_front` makes, with a carried fp32 state
+    ``[lines, n_heads, Dv, D]`` (value channel by key channel).  Per head and step, seen as a matrix ``M`` of key channels by value
+    channels: row ``d`` of ``M`` is multiplied by ``decay[d]``, then ``e = b * (v - M' k)``, ``M += outer(k, e)``, and ``y = M' q``
+    reads the corrected state.  Head ``h`` reads q / k head ``h // (n_heads / n_qk)``.  Returns y fp32 [B, T, n_heads * Dv]; padding
+    steps leave the state untouched."""
+    B, T = qkv.shape[:2]
+    H, rep, Cq = n_heads, n_heads // n_qk, n_qk * D
+    q = qkv[..., :Cq].float().reshape(B, T, n_qk, D).repeat_interleave(rep, 2)
+    k = qkv[..., Cq:2 * Cq].float().reshape(B, T, n_qk, D).repeat_interleave(rep, 2)
+    v = qkv[..., 2 * Cq:].float().reshape(B, T, H, Dv)
+    g = decay.float().reshape(B, T, H, D)
+    S = state[slots.long()].float()
+    S = torch.where((ctx_len > 0).view(B, 1, 1, 1), S, torch.zeros_like(S))
+    out = []
+    for t in range(T):
+        live = (t < q_len).view(B, 1, 1, 1)
+        Sn = S * g[:, t, :, None, :]
+        e = beta[:, t, :, None].float() * (v[:, t] - (Sn * k[:, t, :, None, :]).sum(-1))
+        Sn = Sn + e.unsqueeze(-1) * k[:, t, :, None, :]
+        S = torch.where(live, Sn, S)
+        out.append((S * q[:, t, :, None, :]).sum(-1))
+    state[slots.long()] = torch.where((q_len > 0).view(B, 1, 1, 1), S, state[slots.long()].float()).to(state.dtype)
+    return torch.stack(out, 1).reshape(B, T, H * Dv)
+
+
+def decay_scan(p, decay, state, slots, ctx_len, q_len, n_heads: int, D: int, Dv: int, silu: bool = True):
+    """Linear attention with a fixed decay per head and a carried fp32 state ``[lines, n_heads, Dv, D]``.  ``p`` [B, T, >= n_heads (2 D +
+    Dv)] holds q | k | v projections (SiLU on all of them when ``silu``).  Per head, seen as a matrix of key channels by value channels:
+    ``M <- decay[h] M + outer(k, v)``, ``y = M' q``.  Returns y fp32 [B, T, n_heads * Dv]; padding steps leave the state untouched."""
+    B, T = p.shape[:2]
+    H = n_heads
+    x = p[..., :H * (2 * D + Dv)].float()
+    x = F.silu(x) if silu else x
+    q, k, v = (t.reshape(B, T, H, -1) for t in x.split([H * D, H * D, H * Dv], -1))
+    S = state[slots.long()].float()
+    S = torch.where((ctx_len > 0).view(B, 1, 1, 1), S, torch.zeros_like(S))
+    lam = decay.float().view(1, H, 1, 1)
+    out = []
+    for t in range(T):
+        S = torch.where((t < q_len).view(B, 1, 1, 1), S * lam + v[:, t, :, :, None] * k[:, t, :, None, :], S)
+        out.append((S * q[:, t, :, None, :]).sum(-1))
+    state[slots.long()] = torch.where((q_len > 0).view(B, 1, 1, 1), S, state[slots.long()].float()).to(state.dtype)
+    return torch.stack(out, 1).reshape(B, T, H * Dv)
+
+
+def table_route(table, token_ids, q_len):
+    """Routing by token id: row ``token_ids[b, t]`` of ``table`` [vocab, k] lists the token's experts, each with weight ``1 / k``.
+    ``token_ids`` [B, T]; tokens past ``q_len[b]`` are routed nowhere (expert -1).  Returns (weights [B T, k] fp32, ids [B T, k] int32)."""
+    B, T = token_ids.shape
+    k = table.shape[1]
+    idx = table[token_ids.long()]
+    live = (torch.arange(T, device=token_ids.device).view(1, T) < q_len.long().view(B, 1)).unsqueeze(-1)
+    idx = torch.where(live, idx, torch.full_like(idx, -1)).reshape(B * T, k).to(torch.int32)
+    return torch.full((B * T, k), 1.0 / k, dtype=torch.float32, device=table.device), idx

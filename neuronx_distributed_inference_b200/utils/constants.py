@@ -102,7 +102,8 @@ MODEL_TYPES["fetodra"] = {"causal-lm": f"{_P}.fetodra.modeling_fetodra:NeuronFet
 MODEL_TYPES["sodudra"] = {"causal-lm": f"{_P}.sodudra.modeling_sodudra:NeuronSodudraForCausalLM"}
 MODEL_TYPES["tusipel"] = {"causal-lm": f"{_P}.tusipel.modeling_tusipel:NeuronTusipelForCausalLM"}
 MODEL_TYPES["zanivik"] = {"causal-lm": f"{_P}.zanivik.modeling_zanivik:NeuronZanivikForCausalLM"}
-ARCHITECTURES = {"Fetodra": "fetodra", "Sodudra": "sodudra", "Tusipel": "tusipel", "Zanivik": "zanivik"}
+MODEL_TYPES["balivik"] = {"causal-lm": f"{_P}.balivik.modeling_balivik:NeuronBalivikForCausalLM"}
+ARCHITECTURES = {"Fetodra": "fetodra", "Sodudra": "sodudra", "Tusipel": "tusipel", "Zanivik": "zanivik", "Balivik": "balivik"}
 TASK_TYPES = ("causal-lm", "image-text-to-text", "speech-to-text", "text-to-image", "audio-frame-classification", "audio-text-to-text")
 
 
