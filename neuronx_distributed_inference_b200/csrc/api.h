@@ -95,7 +95,8 @@ void qgemv_launch(const void* x, const void* w, const float* scale, int scale_n,
 
 // MoE decode: routed experts for T <= 8 tokens as two batched streaming launches (moe_decode.cu)
 void moe_decode_launch(const void* x, const void* w_gate_up, const void* w_down, const float* topk_w, const int* topk_i, void* u,
-                       float* y_acc, int T, int topk, int H, int I, int E, int expert_offset, int n_sms, cudaStream_t stream);
+                       float* y_acc, int T, int topk, int H, int I, int E, int expert_offset, int act /*1 silu*up, 4 clamped gate product*/, float limit,
+                       float alpha, int n_sms, cudaStream_t stream);
 
 struct AttnDecodeParams {
   const void* q;        // [B, T, Hq, D] bf16
@@ -152,7 +153,8 @@ void moe_gather_launch(const void* x, const float* topk_w, const int* row_entry,
 void moe_combine_launch(const void* y, const float* topk_w, const int* pos, void* out, int N, int H, int k, int scale_input,
                         cudaStream_t stream);
 void gemm_grouped_launch(const void* a, const void* b, const void* bias, void* c, int R, int N, int K, int n_experts, int act,
-                         const int* tile_expert, const float* a_scale, const float* w_scale, cudaStream_t stream);
+                         const int* tile_expert, const float* a_scale, const float* w_scale, cudaStream_t stream, float glu_limit = 7.f,
+                         float glu_alpha = 1.702f);      // limit, alpha: act 4
 
 // symmetric heap (symm_heap.cpp) and NVLS collectives (nvls.cu)
 long long symm_heap_create(long long bytes, int device, int world, int rank);

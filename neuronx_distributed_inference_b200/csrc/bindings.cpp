@@ -221,7 +221,8 @@ at::Tensor gemv_allreduce(const at::Tensor& x, const at::Tensor& w, const c10::o
 // Routed experts of a decode step: x [T,H], w_gate_up [E,2I,H], w_down [E,H,I], topk_w/topk_i [T,k] -> [T,H] (local experts only;
 // the caller all-reduces across EP/TP ranks).
 at::Tensor moe_decode(const at::Tensor& x, const at::Tensor& w_gate_up, const at::Tensor& w_down, const at::Tensor& topk_w,
-                      const at::Tensor& topk_i, int64_t expert_offset) {
+                      const at::Tensor& topk_i, int64_t expert_offset, int64_t act, double limit, double alpha) {
+  TORCH_CHECK(act == 1 || act == 4, "moe_decode: SiLU or clamped gate product");
   TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.is_contiguous() && is_bf16(x) && is_bf16(w_gate_up) && is_bf16(w_down));
   TORCH_CHECK(w_gate_up.dim() == 3 && w_down.dim() == 3 && w_gate_up.is_contiguous() && w_down.is_contiguous());
   const int T = x.size(0), H = x.size(1), E = w_gate_up.size(0), I = w_gate_up.size(1) / 2, k = topk_i.size(1);
@@ -234,7 +235,7 @@ at::Tensor moe_decode(const at::Tensor& x, const at::Tensor& w_gate_up, const at
   static int n_sms = 0;
   if (n_sms == 0) n_sms = at::cuda::getCurrentDeviceProperties()->multiProcessorCount;
   moe_decode_launch(x.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), topk_w.data_ptr<float>(), topk_i.data_ptr<int>(),
-                    u.data_ptr(), y.data_ptr<float>(), T, k, H, I, E, (int)expert_offset, n_sms, cur_stream());
+                    u.data_ptr(), y.data_ptr<float>(), T, k, H, I, E, (int)expert_offset, (int)act, (float)limit, (float)alpha, n_sms, cur_stream());
   return y.to(x.scalar_type());
 }
 
@@ -256,7 +257,7 @@ at::Tensor dequant_bf16(const at::Tensor& w, const at::Tensor& scale, at::Tensor
 at::Tensor moe_grouped(const at::Tensor& x, const at::Tensor& w_gate_up, const at::Tensor& w_down, const at::Tensor& topk_w,
                        const at::Tensor& topk_i, int64_t expert_offset, int64_t act, bool scale_input,
                        const c10::optional<at::Tensor>& gate_up_bias, const c10::optional<at::Tensor>& down_bias,
-                       const c10::optional<at::Tensor>& gate_up_scale, const c10::optional<at::Tensor>& down_scale) {
+                       const c10::optional<at::Tensor>& gate_up_scale, const c10::optional<at::Tensor>& down_scale, double limit, double alpha) {
   // W8A8 experts: fp8-e4m3 weights with per-(expert, channel) scales; the permuted activations and the intermediate are quantised
   // per row (quant.cu) and both grouped GEMMs run on the kind::f8f6f4 tensor-core path
   const bool fp8 = gate_up_scale.has_value();
@@ -302,13 +303,13 @@ at::Tensor moe_grouped(const at::Tensor& x, const at::Tensor& w_gate_up, const a
     auto xs = at::empty({R}, x.options().dtype(at::kFloat)), hs = at::empty({R}, x.options().dtype(at::kFloat));
     rmsnorm_quant_launch(xp.data_ptr(), nullptr, xq.data_ptr(), xs.data_ptr<float>(), (int)R, H, 0.f, 0.f, inf, st);
     gemm_grouped_launch(xq.data_ptr(), w_gate_up.data_ptr(), gate_up_bias ? gate_up_bias->data_ptr() : nullptr, h.data_ptr(), (int)R, 2 * I,
-                        H, E, (int)act, tile_expert.data_ptr<int>(), xs.data_ptr<float>(), gate_up_scale->data_ptr<float>(), st);
+                        H, E, (int)act, tile_expert.data_ptr<int>(), xs.data_ptr<float>(), gate_up_scale->data_ptr<float>(), st, (float)limit, (float)alpha);
     rmsnorm_quant_launch(h.data_ptr(), nullptr, hq.data_ptr(), hs.data_ptr<float>(), (int)R, I, 0.f, 0.f, inf, st);
     gemm_grouped_launch(hq.data_ptr(), w_down.data_ptr(), down_bias ? down_bias->data_ptr() : nullptr, y.data_ptr(), (int)R, H, I, E, 0,
                         tile_expert.data_ptr<int>(), hs.data_ptr<float>(), down_scale->data_ptr<float>(), st);
   } else {
     gemm_grouped_launch(xp.data_ptr(), w_gate_up.data_ptr(), gate_up_bias ? gate_up_bias->data_ptr() : nullptr, h.data_ptr(), (int)R,
-                        2 * I, H, E, (int)act, tile_expert.data_ptr<int>(), nullptr, nullptr, st);
+                        2 * I, H, E, (int)act, tile_expert.data_ptr<int>(), nullptr, nullptr, st, (float)limit, (float)alpha);
     gemm_grouped_launch(h.data_ptr(), w_down.data_ptr(), down_bias ? down_bias->data_ptr() : nullptr, y.data_ptr(), (int)R, H, I, E, 0,
                         tile_expert.data_ptr<int>(), nullptr, nullptr, st);
   }

@@ -34,7 +34,8 @@ struct GemmParams {
   const __nv_bfloat16* bias;      // [N] or null
   const __nv_bfloat16* residual;  // [M, N_out] or null
   __nv_bfloat16* c;               // [M, N_out]
-  int M, N, K, ldc, act;          // act: 0 none, 1 silu*up, 2 gelu_tanh*up, 3 gelu*up, 4 GPT-OSS clamped SwiGLU  (N_out = N/2 when act != 0)
+  int M, N, K, ldc, act;          // act: 0 none, 1 silu*up, 2 gelu_tanh*up, 3 gelu*up, 4 clamped gate product  (N_out = N/2 when act != 0)
+  float glu_limit, glu_alpha;     // act 4 (GPT-OSS: 7, 1.702)
   int m_tiles, n_tiles;           // tile grid (CTA tiles of TM*128 x 128 output columns; 64 output features for GLU)
   // fp8 (e4m3 x e4m3 -> fp32, tcgen05 kind::f8f6f4): acc * a_scale[row] * w_scale[col] (dynamic per-token activation scale,
   // per-output-channel or per-tensor weight scale); null for bf16
@@ -330,9 +331,9 @@ __global__ void __launch_bounds__(GM_THREADS, 1) gemm_tcgen05_kernel(const __gri
           if (glu) {
             float up = __uint_as_float(vu[j + e]) * up_s;
             if (p.bias && in) up += __bfloat162float(p.bias[cur_eo + n_out + col0 + j + e]);
-            if (p.act == 4) {   // GPT-OSS clamped SwiGLU: (clamp(up, -7, 7) + 1) * g * sigmoid(1.702 g), g = min(gate, 7)
-              const float g = fminf(a, 7.f), u = fminf(fmaxf(up, -7.f), 7.f);
-              a = (u + 1.f) * g * (1.f / (1.f + __expf(-1.702f * g)));
+            if (p.act == 4) {   // clamped gate product: (clamp(up, -limit, limit) + 1) * g * sigmoid(alpha g), g = min(gate, limit)
+              const float g = fminf(a, p.glu_limit), u = fminf(fmaxf(up, -p.glu_limit), p.glu_limit);
+              a = (u + 1.f) * g * (1.f / (1.f + __expf(-p.glu_alpha * g)));
             } else {
               a = (p.act == 1 ? silu(a) : (p.act == 2 ? gelu_tanh(a) : gelu_erf(a))) * up;
             }
@@ -612,7 +613,7 @@ static unsigned* gemm_tickets() {
 
 static void gemm_launch_impl(const void* a, int lda, const void* b, const void* bias, const void* residual, void* c, int ldc, int M, int N,
                              int K, int act, cudaStream_t stream, const GemmRsArgs* rs, const float* a_scale, const float* w_scale,
-                             int w_scale_n, const int* tile_expert = nullptr, int n_experts = 1) {
+                             int w_scale_n, const int* tile_expert = nullptr, int n_experts = 1, float glu_limit = 7.f, float glu_alpha = 1.702f) {
   GemmParams p{};
   p.grp_tile_expert = tile_expert;
   const bool glu = act != 0;
@@ -627,7 +628,7 @@ static void gemm_launch_impl(const void* a, int lda, const void* b, const void* 
   p.bias = reinterpret_cast<const __nv_bfloat16*>(bias);
   p.residual = reinterpret_cast<const __nv_bfloat16*>(residual);
   p.c = reinterpret_cast<__nv_bfloat16*>(c);
-  p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.act = act;
+  p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.act = act; p.glu_limit = glu_limit; p.glu_alpha = glu_alpha;
   // TM = 2 (256-row CTA tiles) whenever there is more than one 128-row block: each weight tile then feeds two UMMAs
   static int force_tm = -1;
   if (force_tm < 0) {
@@ -767,11 +768,11 @@ void gemm_tcgen05_launch(const void* a, int lda, const void* b, const void* bias
 // grouped GEMM of the mixture-of-experts layers: a [R, K] tokens permuted by expert (R % 128 == 0), b [E, N, K] stacked expert
 // weights, tile_expert [R / 128] (device; -1 = unused tile), bias [E, N] or null; fp8 when a_scale != null (w_scale [E, N])
 void gemm_grouped_launch(const void* a, const void* b, const void* bias, void* c, int R, int N, int K, int n_experts, int act,
-                         const int* tile_expert, const float* a_scale, const float* w_scale, cudaStream_t stream) {
+                         const int* tile_expert, const float* a_scale, const float* w_scale, cudaStream_t stream, float glu_limit, float glu_alpha) {
   if (K % (a_scale ? 128 : 64) != 0) throw std::runtime_error("grouped gemm: K must be a multiple of 64 (128 for fp8)");
   const int n_out = act ? N / 2 : N;
   gemm_launch_impl(a, K, b, bias, nullptr, c, n_out, R, N, K, act, stream, nullptr, a_scale, w_scale, a_scale ? N : 0, tile_expert,
-                   n_experts);
+                   n_experts, glu_limit, glu_alpha);
 }
 
 // W8A8 fp8-e4m3 GEMM: a [M, K] fp8 with per-row scale, b [N, K] fp8 with per-channel (w_scale_n == N) or per-tensor (1) scale

@@ -1,0 +1,455 @@
+// Linear recurrences over a matrix state per head with value channels outermost, [Dv, D] (the key channels of a value channel are contiguous):
+//   * the gated delta rule with one decay per head and key channel, and the kernel that makes its rows (convolution, SiLU, unit norms,
+//     decays, write strengths);
+//   * linear attention with a fixed decay per head;
+// and routing by token id.  States, decays, unit norms and everything else inside a recurrence are fp32; compiled WITHOUT fast-math.
+#include <cuda_bf16.h>
+#include <math.h>
+
+#include <stdexcept>
+#include <type_traits>
+
+#include "common.cuh"
+#include "seqmix.h"
+
+namespace nxdi {
+namespace {
+
+template <typename T> __device__ __forceinline__ float ldf1(const T* p);
+template <> __device__ __forceinline__ float ldf1<float>(const float* p) { return *p; }
+template <> __device__ __forceinline__ float ldf1<__nv_bfloat16>(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void stf1(float* p, float v) { *p = v; }
+__device__ __forceinline__ void stf1(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ float sigmoid_acc(float v) { return 1.f / (1.f + expf(-v)); }
+__device__ __forceinline__ float silu_acc(float v) { return v / (1.f + expf(-v)); }
+__device__ __forceinline__ float softplus_acc(float v) { return v > 20.f ? v : log1pf(expf(v)); }
+
+// VEC consecutive values as one access
+template <int VEC> __device__ __forceinline__ void ldvec(const float* p, float* x) {
+  if constexpr (VEC == 4) { const float4 v = *reinterpret_cast<const float4*>(p); x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w; }
+  else x[0] = *p;
+}
+template <int VEC> __device__ __forceinline__ void ldvec(const __nv_bfloat16* p, float* x) {
+  if constexpr (VEC == 4) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    x[0] = bf16lo(r.x); x[1] = bf16hi(r.x); x[2] = bf16lo(r.y); x[3] = bf16hi(r.y);
+  } else x[0] = __bfloat162float(*p);
+}
+template <int VEC> __device__ __forceinline__ void stvec(float* p, const float* x) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+  else *p = x[0];
+}
+template <int VEC> __device__ __forceinline__ void stvec(__nv_bfloat16* p, const float* x) {
+  if constexpr (VEC == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]));
+  else *p = __float2bfloat16_rn(x[0]);
+}
+
+// ---- rows of the per-channel delta rule -------------------------------------------------------------------------------------------------
+// A warp takes one segment of channels over a tile of tokens: a q or k head (unit norm), a run of v channels, a run of decays, or all write
+// strengths.  The convolution's window stays in registers while the warp marches over its tokens; only the first tile of a row reads the
+// carried rows, and it writes them back at the end (from the projection rows themselves), so no other warp touches them.
+constexpr int FRONT_WARPS = 8;
+template <typename T, int VEC, int NI, int KM>
+__global__ void __launch_bounds__(FRONT_WARPS * 32) delta_front_kernel(DeltaFrontParams p, int TT, int vsegs, int gsegs) {
+  constexpr int SEG = 32 * VEC * NI, N = VEC * NI;
+  const int b = blockIdx.z, t0 = blockIdx.x * TT, lane = threadIdx.x & 31;
+  const int seg = blockIdx.y * FRONT_WARPS + (threadIdx.x >> 5);
+  const int qn = p.q_len[b], live = min(t0 + TT, qn);
+  if (t0 >= qn) return;
+  const int K = p.K, D = p.D, Cq = p.n_qk * D, Cv = p.nh * p.Dv, C = 2 * Cq + Cv, Cg = p.nh * D;
+  const long long row0 = (long long)b * p.T;
+  if (seg < 2 * p.n_qk + vsegs) {
+    const bool unit = seg < 2 * p.n_qk, isq = seg < p.n_qk;
+    const int first = unit ? seg * D : 2 * Cq + (seg - 2 * p.n_qk) * SEG;              // channel of the row
+    const int width = unit ? D : min(SEG, C - first);
+    const T* src = (const T*)p.p + (long long)b * p.p_sb + first;
+    float ring[KM - 1 > 0 ? KM - 1 : 1][N], cw[KM][N], x[N];
+    bool in[NI];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = (i * 32 + lane) * VEC;
+      in[i] = c < width;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e)
+#pragma unroll
+        for (int d = 0; d < KM; ++d) cw[d][i * VEC + e] = (in[i] && d < K) ? p.conv_w[(long long)(first + c + e) * K + (K - 1 - d)] : 0.f;
+    }
+    T* state = K > 1 ? (T*)p.state + (long long)p.lines[b] * (K - 1) * C + first : nullptr;
+    const bool carried = K > 1 && p.ctx_len[b] > 0;
+    auto load = [&](const T* row, float* dst, bool on) {
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        if (in[i] && on) ldvec<VEC>(row + (i * 32 + lane) * VEC, dst + i * VEC);
+        else
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) dst[i * VEC + e] = 0.f;
+      }
+    };
+    // ring[d]: the input of d + 1 tokens ago
+#pragma unroll
+    for (int d = 0; d < KM - 1; ++d) {
+      const int t = t0 - 1 - d;
+      if (d >= K - 1) load(src, ring[d], false);
+      else if (t >= 0) load(src + (long long)t * p.p_st, ring[d], true);
+      else load(K > 1 ? state + (long long)(K - 1 + t) * C : src, ring[d], carried);
+    }
+    const float qmul = isq ? 1.f / sqrtf((float)D) : 1.f;
+    load(src + (long long)t0 * p.p_st, x, true);
+    for (int t = t0; t < live; ++t) {
+      float y[N], ss = 0.f, cur[N];
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        cur[i] = x[i];
+        float a = cw[0][i] * x[i];
+#pragma unroll
+        for (int d = 1; d < KM; ++d) a += cw[d][i] * ring[d - 1][i];
+        y[i] = silu_acc(a);
+        ss += y[i] * y[i];
+      }
+      if (t + 1 < live) load(src + (long long)(t + 1) * p.p_st, x, true);
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+#pragma unroll
+        for (int d = KM - 2; d > 0; --d) ring[d][i] = ring[d - 1][i];
+        if (KM > 1) ring[0][i] = cur[i];
+      }
+      if (unit) {
+        const float r = qmul / sqrtf(warp_sum(ss) + p.unit_eps);
+#pragma unroll
+        for (int i = 0; i < N; ++i) y[i] *= r;
+      }
+      float* out = p.qkv + (row0 + t) * C + first;
+#pragma unroll
+      for (int i = 0; i < NI; ++i)
+        if (in[i]) stvec<VEC>(out + (i * 32 + lane) * VEC, y + i * VEC);
+    }
+    if (t0 == 0 && K > 1) {
+      // the last K - 1 inputs of (carried rows, this portion); oldest first, so a carried row is read before its place is overwritten
+      for (int j = 0; j < K - 1; ++j) {
+        const int t = qn - (K - 1) + j;
+        float v[N];
+        if (t >= 0) load(src + (long long)t * p.p_st, v, true);
+        else load(state + (long long)(K - 1 + t) * C, v, carried);
+#pragma unroll
+        for (int i = 0; i < NI; ++i)
+          if (in[i]) stvec<VEC>(state + (long long)j * C + (i * 32 + lane) * VEC, v + i * VEC);
+      }
+    }
+  } else if (seg < 2 * p.n_qk + vsegs + gsegs) {
+    const int first = (seg - 2 * p.n_qk - vsegs) * SEG;
+    float nA[N], dt[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int c = first + (i / VEC * 32 + lane) * VEC + i % VEC;
+      nA[i] = c < Cg ? -expf(p.A_log[c / D]) : 0.f;
+      dt[i] = c < Cg ? p.dt_bias[c] : 0.f;
+    }
+    for (int t = t0; t < live; ++t) {
+      const T* src = (const T*)p.a_raw + (long long)b * p.a_sb + (long long)t * p.a_st + first;
+      float* out = p.decay + (row0 + t) * Cg + first;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int c = (i * 32 + lane) * VEC;
+        if (first + c < Cg) {
+          float v[VEC];
+          ldvec<VEC>(src + c, v);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) v[e] = expf(nA[i * VEC + e] * softplus_acc(v[e] + dt[i * VEC + e]));
+          stvec<VEC>(out + c, v);
+        }
+      }
+    }
+  } else if (seg == 2 * p.n_qk + vsegs + gsegs) {
+    for (int t = t0; t < live; ++t)
+      for (int h = lane; h < p.nh; h += 32)
+        p.beta[(row0 + t) * p.nh + h] = sigmoid_acc(ldf1((const T*)p.b_raw + (long long)b * p.b_sb + (long long)t * p.b_st + h));
+  }
+}
+
+// ---- recurrent form ---------------------------------------------------------------------------------------------------------------------
+// Block = (batch row, head, 16 value channels).  A thread holds two value channels and, of each, the key channels j * 32 + ns * 4 .. + 3 (ns = its
+// place among eight lanes), so a lane's 16-byte shared-memory reads of k / q / decay serve both channels, the eight lanes read 128 contiguous
+// bytes, and the state moves in 16-byte pieces.  Time runs in rounds of 16 steps; the rows of the next round land in a second shared-memory
+// stage (cp.async) meanwhile.
+//   delta: s <- decay * s per key channel; r = s . k, o = s . q on the shrunk state share one lane reduction; u = beta (v - r); s += u k;
+//          o += u (k . q), k . q formed once per step and round
+//   fixed: s <- decay_h s + v k;  o = s . q
+constexpr int LS_PT = 16, LS_TT = 16, LS_NS = 8, LS_CPT = 2, LS_THREADS = (LS_PT / LS_CPT) * LS_NS;
+
+template <typename T, bool DELTA, int NJ, bool ALIGNED>
+__global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParams p) {
+  extern __shared__ __align__(16) float lsm[];
+  constexpr int DP = NJ * 32, ROWS = DELTA ? 3 : 2, STAGE = ROWS * LS_TT * DP + LS_TT * LS_PT;
+  float* kq = lsm + 2 * STAGE;                  // [TT] k . q
+  float* bt = kq + LS_TT;                       // [TT] beta
+  float* os = bt + LS_TT;                       // [TT][PT]
+  const int D = p.D, Dv = p.Dv, b = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * LS_PT;
+  const int n_tok = p.q_len[b];
+  if (n_tok <= 0) return;
+  const int tid = threadIdx.x, pl = tid / LS_NS, ns = tid % LS_NS;
+  const int gq = h / (p.nh / p.n_qk), Cq = p.n_qk * D;
+  float* Sg = p.state + ((long long)p.lines[b] * p.nh + h) * Dv * D;
+  const bool has_ctx = p.ctx_len[b] > 0;
+  float4 S[LS_CPT][NJ];
+#pragma unroll
+  for (int c = 0; c < LS_CPT; ++c)
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int d = j * 32 + ns * 4, pc = p0 + pl * LS_CPT + c;
+      S[c][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (has_ctx && pc < Dv) {
+        const float* s = Sg + (long long)pc * D + d;
+        if (ALIGNED) { if (d < D) S[c][j] = *reinterpret_cast<const float4*>(s); }
+        else {
+          if (d < D) S[c][j].x = s[0];
+          if (d + 1 < D) S[c][j].y = s[1];
+          if (d + 2 < D) S[c][j].z = s[2];
+          if (d + 3 < D) S[c][j].w = s[3];
+        }
+      }
+    }
+  const T* xrow = (const T*)p.x + (long long)b * p.x_sb;
+  const float lam = DELTA ? 0.f : p.decay[h];
+  // rows of steps t0 .. into stage st; zeros past the key channels and past the live steps
+  auto issue = [&](int t0, int st) {
+    const int tt = min(LS_TT, n_tok - t0);
+    float* qd = lsm + st * STAGE;
+    float* kd = qd + LS_TT * DP;
+    float* gd = kd + LS_TT * DP;                // delta only
+    float* vd = qd + ROWS * LS_TT * DP;
+    if constexpr (DELTA && ALIGNED) {
+      constexpr int CPR = DP / 4;
+      for (int i = tid; i < LS_TT * CPR; i += LS_THREADS) {
+        const int t = i / CPR, d = (i % CPR) * 4, at = t * DP + d;
+        const bool on = t < tt && d < D;
+        const float* q = on ? (const float*)xrow + (long long)(t0 + t) * p.x_st + gq * D + d : (const float*)xrow;
+        cp_async16(qd + at, q, on);
+        cp_async16(kd + at, on ? q + Cq : q, on);
+        cp_async16(gd + at, on ? p.decay + ((long long)b * p.T + t0 + t) * p.nh * D + h * D + d : (const float*)xrow, on);
+      }
+      for (int i = tid; i < LS_TT * (LS_PT / 4); i += LS_THREADS) {
+        const int t = i / (LS_PT / 4), c = (i % (LS_PT / 4)) * 4;
+        const bool on = t < tt && p0 + c < Dv;
+        cp_async16(vd + t * LS_PT + c, on ? (const float*)xrow + (long long)(t0 + t) * p.x_st + 2 * Cq + h * Dv + p0 + c : (const float*)xrow, on);
+      }
+      cp_async_commit();
+    } else {
+      auto act = [&](float v) { return (!DELTA && p.silu) ? silu_acc(v) : v; };
+      const int tl = (t0 == 0 && tt < LS_TT) ? tt : LS_TT;          // a lone short round touches its live steps only
+      for (int i = tid; i < tl * DP; i += LS_THREADS) {
+        const int t = i / DP, d = i % DP;
+        const bool on = t < tt && d < D;
+        const T* r = xrow + (long long)(t0 + t) * p.x_st + gq * D + d;
+        qd[i] = on ? act(ldf1(r)) : 0.f;
+        kd[i] = on ? act(ldf1(r + Cq)) : 0.f;
+        if (DELTA) gd[i] = on ? p.decay[((long long)b * p.T + t0 + t) * p.nh * D + h * D + d] : 0.f;
+      }
+      for (int i = tid; i < tl * LS_PT; i += LS_THREADS) {
+        const int t = i / LS_PT, c = p0 + i % LS_PT;
+        vd[i] = (t < tt && c < Dv) ? act(ldf1(xrow + (long long)(t0 + t) * p.x_st + 2 * Cq + h * Dv + c)) : 0.f;
+      }
+    }
+  };
+  issue(0, 0);
+  int st = 0;
+  for (int t0 = 0; t0 < n_tok; t0 += LS_TT, st ^= 1) {
+    const int tt = min(LS_TT, n_tok - t0);
+    if constexpr (DELTA && ALIGNED) cp_async_wait<0>();
+    __syncthreads();                            // this round has landed; everyone is done with the other stage, kq, bt and os
+    const float* qs = lsm + st * STAGE;
+    const float* ks = qs + LS_TT * DP;
+    const float* gs = ks + LS_TT * DP;
+    const float* vs = qs + ROWS * LS_TT * DP;
+    if constexpr (DELTA) {
+      // four threads per step form k . q
+      const int t = tid / 4, part = tid % 4;
+      float s = 0.f;
+      if (t < tt) {
+#pragma unroll
+        for (int j = 0; j < NJ * 2; ++j) {
+          const int at = t * DP + (j * 4 + part) * 4;
+          const float4 a = *reinterpret_cast<const float4*>(qs + at), k = *reinterpret_cast<const float4*>(ks + at);
+          s += (a.x * k.x + a.z * k.z) + (a.y * k.y + a.w * k.w);
+        }
+      }
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      s += __shfl_xor_sync(0xffffffffu, s, 2);
+      if (part == 0 && t < tt) {
+        kq[t] = s;
+        bt[t] = p.beta[((long long)b * p.T + t0 + t) * p.nh + h];
+      }
+      __syncthreads();
+    }
+    if (t0 + LS_TT < n_tok) issue(t0 + LS_TT, st ^ 1);
+#pragma unroll 1
+    for (int t = 0; t < tt; ++t) {
+      const float4* Kt = reinterpret_cast<const float4*>(ks + t * DP) + ns;
+      const float4* Qt = reinterpret_cast<const float4*>(qs + t * DP) + ns;
+      float4 kv[NJ];
+      float sq[LS_CPT], vt[LS_CPT];
+#pragma unroll
+      for (int c = 0; c < LS_CPT; ++c) { sq[c] = 0.f; vt[c] = vs[t * LS_PT + pl * LS_CPT + c]; }
+      if constexpr (DELTA) {
+        const float4* Gt = reinterpret_cast<const float4*>(gs + t * DP) + ns;
+        float sk[LS_CPT];
+#pragma unroll
+        for (int c = 0; c < LS_CPT; ++c) sk[c] = 0.f;
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          kv[j] = Kt[j * 8];
+          const float4 qv = Qt[j * 8], gv = Gt[j * 8];
+#pragma unroll
+          for (int c = 0; c < LS_CPT; ++c) {
+            S[c][j].x *= gv.x; S[c][j].y *= gv.y; S[c][j].z *= gv.z; S[c][j].w *= gv.w;
+            sk[c] += (S[c][j].x * kv[j].x + S[c][j].z * kv[j].z) + (S[c][j].y * kv[j].y + S[c][j].w * kv[j].w);
+            sq[c] += (S[c][j].x * qv.x + S[c][j].z * qv.z) + (S[c][j].y * qv.y + S[c][j].w * qv.w);
+          }
+        }
+#pragma unroll
+        for (int o = LS_NS / 2; o > 0; o >>= 1)
+#pragma unroll
+          for (int c = 0; c < LS_CPT; ++c) {
+            sk[c] += __shfl_xor_sync(0xffffffffu, sk[c], o);
+            sq[c] += __shfl_xor_sync(0xffffffffu, sq[c], o);
+          }
+        const float be = bt[t], kqt = kq[t];
+#pragma unroll
+        for (int c = 0; c < LS_CPT; ++c) {
+          const float u = be * (vt[c] - sk[c]);
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) { S[c][j].x += u * kv[j].x; S[c][j].y += u * kv[j].y; S[c][j].z += u * kv[j].z; S[c][j].w += u * kv[j].w; }
+          sq[c] += u * kqt;
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const float4 k4 = Kt[j * 8], qv = Qt[j * 8];
+#pragma unroll
+          for (int c = 0; c < LS_CPT; ++c) {
+            S[c][j].x = lam * S[c][j].x + vt[c] * k4.x; S[c][j].y = lam * S[c][j].y + vt[c] * k4.y;
+            S[c][j].z = lam * S[c][j].z + vt[c] * k4.z; S[c][j].w = lam * S[c][j].w + vt[c] * k4.w;
+            sq[c] += (S[c][j].x * qv.x + S[c][j].z * qv.z) + (S[c][j].y * qv.y + S[c][j].w * qv.w);
+          }
+        }
+#pragma unroll
+        for (int o = LS_NS / 2; o > 0; o >>= 1)
+#pragma unroll
+          for (int c = 0; c < LS_CPT; ++c) sq[c] += __shfl_xor_sync(0xffffffffu, sq[c], o);
+      }
+      if (ns == 0)
+#pragma unroll
+        for (int c = 0; c < LS_CPT; ++c) os[t * LS_PT + pl * LS_CPT + c] = sq[c];
+    }
+    __syncthreads();
+    for (int i = tid; i < tt * LS_PT; i += LS_THREADS) {
+      const int t = i / LS_PT, c = p0 + i % LS_PT;
+      if (c < Dv) p.y[((long long)b * p.T + t0 + t) * p.nh * Dv + h * Dv + c] = os[i];
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < LS_CPT; ++c)
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int d = j * 32 + ns * 4, pc = p0 + pl * LS_CPT + c;
+      if (pc < Dv) {
+        float* s = Sg + (long long)pc * D + d;
+        if (ALIGNED) { if (d < D) *reinterpret_cast<float4*>(s) = S[c][j]; }
+        else {
+          if (d < D) s[0] = S[c][j].x;
+          if (d + 1 < D) s[1] = S[c][j].y;
+          if (d + 2 < D) s[2] = S[c][j].z;
+          if (d + 3 < D) s[3] = S[c][j].w;
+        }
+      }
+    }
+}
+
+__global__ void __launch_bounds__(256) table_route_kernel(const int* __restrict__ table, const int* __restrict__ ids, const int* __restrict__ q_len,
+                                                          float* __restrict__ w, int* __restrict__ idx, int B, int T, int k, int vocab) {
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= (long long)B * T * k) return;
+  const long long tok = i / k;
+  const int id = ids[tok];
+  const bool on = (int)(tok % T) < q_len[tok / T] && id >= 0 && id < vocab;
+  idx[i] = on ? table[(long long)id * k + i % k] : -1;
+  w[i] = 1.f / (float)k;
+}
+
+template <typename K>
+void opt_in(K kernel, size_t bytes) {
+  if (bytes > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+}
+
+template <typename T, bool DELTA>
+void scan_go(const LinearScanParams& p, bool aligned, cudaStream_t st) {
+  const dim3 grid((p.Dv + LS_PT - 1) / LS_PT, p.nh, p.B);
+  auto go = [&](auto nj, auto al) {
+    constexpr int NJ = decltype(nj)::value;
+    constexpr bool AL = decltype(al)::value;
+    constexpr size_t stage = (DELTA ? 3 : 2) * LS_TT * NJ * 32 + LS_TT * LS_PT;
+    const size_t smem = sizeof(float) * (2 * stage + 2 * LS_TT + LS_TT * LS_PT);
+    auto kernel = linear_scan_kernel<T, DELTA, NJ, AL>;
+    opt_in(kernel, smem);
+    kernel<<<grid, LS_THREADS, smem, st>>>(p);
+  };
+  auto by_size = [&](auto al) {
+    if (p.D <= 64) go(std::integral_constant<int, 2>{}, al);
+    else if (p.D <= 128) go(std::integral_constant<int, 4>{}, al);
+    else go(std::integral_constant<int, 8>{}, al);
+  };
+  if (aligned) by_size(std::true_type{}); else by_size(std::false_type{});
+}
+
+}  // namespace
+
+void delta_front_launch(const DeltaFrontParams& p, bool lp, cudaStream_t st) {
+  if (p.B <= 0 || p.T <= 0) return;
+  if (p.D > 256 || p.K > SEQMIX_MAX_TAPS || p.nh % p.n_qk != 0) throw std::runtime_error("delta_front: key size <= 256, taps <= 8, heads a multiple of q / k heads");
+  const int C = 2 * p.n_qk * p.D + p.nh * p.Dv, Cg = p.nh * p.D;
+  const size_t va = lp ? 8 : 16, esz = lp ? 2 : 4;
+  auto al = [&](const void* q) { return ((uintptr_t)q % va) == 0; };
+  const bool vec = p.D % 4 == 0 && C % 4 == 0 && al(p.p) && al(p.a_raw) && al(p.state) && (p.p_sb * esz) % va == 0 && (p.p_st * esz) % va == 0 &&
+                   (p.a_sb * esz) % va == 0 && (p.a_st * esz) % va == 0 && ((uintptr_t)p.qkv % 16) == 0 && ((uintptr_t)p.decay % 16) == 0;
+  auto go = [&](auto tag, auto ve, auto ni, auto km) {
+    using T = decltype(tag);
+    constexpr int VEC = decltype(ve)::value, NI = decltype(ni)::value, KM = decltype(km)::value, SEG = 32 * VEC * NI;
+    // tiles hold at least K - 1 tokens: only the first one of a row needs the carried rows
+    const int TT = p.T == 1 ? 1 : 8;
+    const int vsegs = (p.nh * p.Dv + SEG - 1) / SEG, gsegs = (Cg + SEG - 1) / SEG, segs = 2 * p.n_qk + vsegs + gsegs + 1;
+    const dim3 grid((p.T + TT - 1) / TT, (segs + FRONT_WARPS - 1) / FRONT_WARPS, p.B);
+    delta_front_kernel<T, VEC, NI, KM><<<grid, FRONT_WARPS * 32, 0, st>>>(p, TT, vsegs, gsegs);
+  };
+  using std::integral_constant;
+  auto by_taps = [&](auto tag, auto ve, auto ni) {
+    if (p.K <= 4) go(tag, ve, ni, integral_constant<int, 4>{}); else go(tag, ve, ni, integral_constant<int, 8>{});
+  };
+  auto by_size = [&](auto tag) {
+    if (vec && p.D <= 128) by_taps(tag, integral_constant<int, 4>{}, integral_constant<int, 1>{});
+    else if (vec) by_taps(tag, integral_constant<int, 4>{}, integral_constant<int, 2>{});
+    else by_taps(tag, integral_constant<int, 1>{}, integral_constant<int, 8>{});
+  };
+  if (lp) by_size(__nv_bfloat16{}); else by_size(float{});
+}
+
+void channel_delta_scan_launch(const LinearScanParams& p, cudaStream_t st) {
+  if (p.B <= 0 || p.T <= 0) return;
+  if (p.D > 256 || p.nh % p.n_qk != 0) throw std::runtime_error("channel_delta_scan: key size <= 256, heads a multiple of q / k heads");
+  const bool aligned = p.D % 4 == 0 && p.Dv % 4 == 0 && p.x_st % 4 == 0 && p.x_sb % 4 == 0 &&
+                       (((uintptr_t)p.x | (uintptr_t)p.decay | (uintptr_t)p.state) & 15) == 0;
+  scan_go<float, true>(p, aligned, st);
+}
+
+void decay_scan_launch(const LinearScanParams& p, bool lp, cudaStream_t st) {
+  if (p.B <= 0 || p.T <= 0) return;
+  if (p.D > 256 || p.n_qk != p.nh) throw std::runtime_error("decay_scan: key size <= 256");
+  const bool aligned = p.D % 4 == 0 && ((uintptr_t)p.state & 15) == 0;
+  if (lp) scan_go<__nv_bfloat16, false>(p, aligned, st); else scan_go<float, false>(p, aligned, st);
+}
+
+void table_route_launch(const int* table, const int* ids, const int* q_len, float* w, int* idx, int B, int T, int k, int vocab, cudaStream_t st) {
+  const long long n = (long long)B * T * k;
+  if (n <= 0) return;
+  table_route_kernel<<<(unsigned)((n + 255) / 256), 256, 0, st>>>(table, ids, q_len, w, idx, B, T, k, vocab);
+}
+
+}  // namespace nxdi

@@ -25,7 +25,7 @@ __global__ void __launch_bounds__(MOE_THREADS) moe_rows_kernel(const __nv_bfloat
                                                                 const float* __restrict__ topk_w,         // [P] (K2 only)
                                                                 __nv_bfloat16* __restrict__ u_out,        // K1: [P, N]
                                                                 float* __restrict__ y_acc,                // K2: [T, N] fp32 (atomics)
-                                                                int K, int N, int topk, int E, int expert_offset) {
+                                                                int K, int N, int topk, int E, int expert_offset, int act, float limit, float alpha) {
   extern __shared__ __align__(16) uint8_t smem[];
   uint4* xs = reinterpret_cast<uint4*>(smem);
   pdl_launch_dependents();
@@ -71,14 +71,22 @@ __global__ void __launch_bounds__(MOE_THREADS) moe_rows_kernel(const __nv_bfloat
     acc_a = warp_sum(acc_a);
     if (GLU) acc_b = warp_sum(acc_b);
     if (lane == 0) {
-      if (GLU) u_out[(size_t)p * N + r] = __float2bfloat16(silu(acc_a) * acc_b);
+      if (GLU) {
+        float u = silu(acc_a) * acc_b;
+        if (act == 4) {      // clamped, shifted gate product
+          const float g = fminf(acc_a, limit);
+          u = g / (1.f + __expf(-alpha * g)) * (fminf(fmaxf(acc_b, -limit), limit) + 1.f);
+        }
+        u_out[(size_t)p * N + r] = __float2bfloat16(u);
+      }
       else atomicAdd(y_acc + (size_t)t * N + r, topk_w[p] * acc_a);
     }
   }
 }
 
 void moe_decode_launch(const void* x, const void* w_gate_up, const void* w_down, const float* topk_w, const int* topk_i, void* u,
-                       float* y_acc, int T, int topk, int H, int I, int E, int expert_offset, int n_sms, cudaStream_t stream) {
+                       float* y_acc, int T, int topk, int H, int I, int E, int expert_offset, int act, float limit, float alpha, int n_sms,
+                       cudaStream_t stream) {
   const int P = T * topk;
   if (H % 8 != 0 || I % 8 != 0) throw std::runtime_error("moe_decode: H and I must be multiples of 8");
   const int gx = std::max(1, (4 * n_sms + P - 1) / P);
@@ -93,10 +101,10 @@ void moe_decode_launch(const void* x, const void* w_gate_up, const void* w_down,
   if ((size_t)H * 2 > 64 * 1024 || (size_t)I * 2 > 64 * 1024) throw std::runtime_error("moe_decode: row too wide for shared memory");
   launch_pdl(k1, dim3(std::min(gx, I), P), dim3(MOE_THREADS), (size_t)H * 2, stream, reinterpret_cast<const __nv_bfloat16*>(x),
              reinterpret_cast<const __nv_bfloat16*>(w_gate_up), topk_i, topk_w, reinterpret_cast<__nv_bfloat16*>(u),
-             static_cast<float*>(nullptr), H, I, topk, E, expert_offset);
+             static_cast<float*>(nullptr), H, I, topk, E, expert_offset, act, limit, alpha);
   launch_pdl(k2, dim3(std::min(gx, H), P), dim3(MOE_THREADS), (size_t)I * 2, stream, reinterpret_cast<const __nv_bfloat16*>(u),
              reinterpret_cast<const __nv_bfloat16*>(w_down), topk_i, topk_w, static_cast<__nv_bfloat16*>(nullptr), y_acc, I, H, topk,
-             E, expert_offset);
+             E, expert_offset, act, limit, alpha);
 }
 
 }  // namespace nxdi

@@ -39,6 +39,15 @@ __device__ __forceinline__ float act_apply(int act, float v) {
   }
 }
 
+constexpr int ACT_CLAMPED_GLU = 7;
+// hidden value of a gated expert: act(g) * u, or the clamped, shifted gate product
+__device__ __forceinline__ float gate_product(int act, float g, float u, float limit, float alpha) {
+  if (act != ACT_CLAMPED_GLU) return act_apply(act, g) * u;
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128) gather_kernel(const T* __restrict__ x, const int* __restrict__ row_entry,
                                                      const int* __restrict__ tile_expert, T* __restrict__ xp, int H, int k) {
@@ -142,7 +151,7 @@ __device__ __forceinline__ float warp_dot(const T* a, const T* b, int n, int lan
 template <typename T>
 __global__ void __launch_bounds__(256) decode_up_kernel(const T* __restrict__ x, const T* __restrict__ w_up, const int* __restrict__ topk_i,
                                                         T* __restrict__ h, int entries, int k, int H, int I, int expert_offset, int e_local,
-                                                        int act, int gated) {
+                                                        int act, int gated, float limit, float alpha) {
   const int lane = threadIdx.x & 31;
   const long long wid = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (wid >= (long long)entries * I) return;
@@ -156,7 +165,7 @@ __global__ void __launch_bounds__(256) decode_up_kernel(const T* __restrict__ x,
       g = __bfloat162float(__float2bfloat16_rn(g));
       u = __bfloat162float(__float2bfloat16_rn(u));
     }
-    if (lane == 0) stx(h + (size_t)ent * I + i, act_apply(act, g) * u);
+    if (lane == 0) stx(h + (size_t)ent * I + i, gate_product(act, g, u, limit, alpha));
     return;
   }
   const float v = warp_dot(x + (size_t)(ent / k) * H, w_up + ((size_t)e * I + i) * H, H, lane);
@@ -352,12 +361,12 @@ __global__ void __launch_bounds__(256) router_select_kernel(const float* __restr
 
 // gated experts: h[r, i] = act(g[r, i]) * g[r, I + i] for the rows of used tiles of the [R, 2 I] first product
 template <typename T>
-__global__ void __launch_bounds__(256) gate_mul_rows_kernel(const T* __restrict__ gu, T* __restrict__ h, int I, int act,
-                                                            const int* __restrict__ tile_expert) {
+__global__ void __launch_bounds__(256) gate_mul_rows_kernel(const T* __restrict__ gu, T* __restrict__ h, int I, int act, float limit,
+                                                            float alpha, const int* __restrict__ tile_expert) {
   const int r = blockIdx.x;
   if (tile_expert[r >> 7] < 0) return;
   const T* row = gu + (size_t)r * 2 * I;
-  for (int i = threadIdx.x; i < I; i += 256) stx(h + (size_t)r * I + i, act_apply(act, ldx(row + i)) * ldx(row + I + i));
+  for (int i = threadIdx.x; i < I; i += 256) stx(h + (size_t)r * I + i, gate_product(act, ldx(row + i), ldx(row + I + i), limit, alpha));
 }
 
 }  // namespace
@@ -408,24 +417,26 @@ void moe_plain_combine_launch(const void* y, const float* topk_w, const int* pos
   else combine_kernel<float><<<N, 128, 0, st>>>((const float*)y, topk_w, pos, (float*)out, H, k);
 }
 
-void moe_plain_gate_mul_launch(const void* gu, void* h, int R, int I, int act, const int* tile_expert, bool lp, cudaStream_t st) {
+void moe_plain_gate_mul_launch(const void* gu, void* h, int R, int I, int act, float limit, float alpha, const int* tile_expert, bool lp,
+                               cudaStream_t st) {
   if (R <= 0) return;
-  if (lp) gate_mul_rows_kernel<__nv_bfloat16><<<R, 256, 0, st>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)h, I, act, tile_expert);
-  else gate_mul_rows_kernel<float><<<R, 256, 0, st>>>((const float*)gu, (float*)h, I, act, tile_expert);
+  if (lp) gate_mul_rows_kernel<__nv_bfloat16><<<R, 256, 0, st>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)h, I, act, limit, alpha, tile_expert);
+  else gate_mul_rows_kernel<float><<<R, 256, 0, st>>>((const float*)gu, (float*)h, I, act, limit, alpha, tile_expert);
 }
 
 void moe_plain_decode_launch(const void* x, const void* w_up, const void* w_down, const float* topk_w, const int* topk_i, void* h, void* out,
-                             int N, int k, int H, int I, int expert_offset, int e_local, int act, bool gated, bool lp, cudaStream_t st) {
+                             int N, int k, int H, int I, int expert_offset, int e_local, int act, bool gated, float limit, float alpha, bool lp,
+                             cudaStream_t st) {
   if (N <= 0) return;
   const long long w1 = (long long)N * k * I, w2 = (long long)N * H;
   const unsigned g1 = (unsigned)((w1 + 7) / 8), g2 = (unsigned)((w2 + 7) / 8);
   if (lp) {
     decode_up_kernel<__nv_bfloat16><<<g1, 256, 0, st>>>((const __nv_bfloat16*)x, (const __nv_bfloat16*)w_up, topk_i, (__nv_bfloat16*)h, N * k, k, H, I,
-                                                        expert_offset, e_local, act, (int)gated);
+                                                        expert_offset, e_local, act, (int)gated, limit, alpha);
     decode_down_kernel<__nv_bfloat16><<<g2, 256, 0, st>>>((const __nv_bfloat16*)h, (const __nv_bfloat16*)w_down, topk_w, topk_i, (__nv_bfloat16*)out, N, k,
                                                           H, I, expert_offset, e_local);
   } else {
-    decode_up_kernel<float><<<g1, 256, 0, st>>>((const float*)x, (const float*)w_up, topk_i, (float*)h, N * k, k, H, I, expert_offset, e_local, act, (int)gated);
+    decode_up_kernel<float><<<g1, 256, 0, st>>>((const float*)x, (const float*)w_up, topk_i, (float*)h, N * k, k, H, I, expert_offset, e_local, act, (int)gated, limit, alpha);
     decode_down_kernel<float><<<g2, 256, 0, st>>>((const float*)h, (const float*)w_down, topk_w, topk_i, (float*)out, N, k, H, I, expert_offset,
                                                   e_local);
   }

@@ -255,11 +255,13 @@ __device__ __forceinline__ float dot_row(const float* qs, const T* k, int D, boo
 constexpr int ATT_WARPS = 4;
 constexpr int ATT_VPL = SEQMIX_MAX_VDIM / 32;      // value channels per lane
 
-// SPLIT = false: warp w of a block owns query blockIdx.x * 4 + w.  SPLIT = true: the four warps share query blockIdx.x, warp w takes
+// SPLIT = false: warp w of a block owns query blockIdx.x * 4 + w.  SPLIT = true: the warps share query blockIdx.x, warp w takes
 // key chunks w, w + 4, ... and the partial (max, sum, acc) are merged through shared memory (few queries, long ranges: decode).
-template <typename T, bool SPLIT>
+// MAPS = 2 (differential attention): a head has two queries and two keys per token over the same values; a query's warp attends with one
+// after the other (SPLIT: half of the warps with each), and the epilogue subtracts, normalises and scales.
+template <typename T, bool SPLIT, int MAPS>
 __global__ void __launch_bounds__(SPLIT ? 1024 : ATT_WARPS * 32) paged_window_attention_kernel(WindowAttnParams p) {
-  extern __shared__ float smem[];      // [warps][D] scaled queries, then (SPLIT) [warps][Dv + 2] partials
+  extern __shared__ float smem[];      // [warps][D] scaled queries, then [warps][Dv + 2] partials
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
   const long long nq = (long long)p.B * p.T * p.Hq;
   const long long qi = SPLIT ? (long long)blockIdx.x : (long long)blockIdx.x * nwarps + warp;
@@ -268,14 +270,10 @@ __global__ void __launch_bounds__(SPLIT ? 1024 : ATT_WARPS * 32) paged_window_at
   const long long tok = in_range ? qi / p.Hq : 0;
   const int b = (int)(tok / p.T), t = (int)(tok % p.T);
   const bool live = in_range && t < p.q_len[b];
-  if (!SPLIT && !live) return;
-  if (SPLIT && !live) return;          // uniform over the block: all warps share the query
+  if (!live) return;                   // SPLIT: uniform over the block, all warps share the query
   const int D = p.D, Dv = p.Dv, g = h / (p.Hq / p.G);
   float* qs = smem + warp * D;
-  const T* qrow = (const T*)p.q + qi * D;
   const float qscale = p.head_scale ? p.scale * p.head_scale[h] : p.scale;
-  for (int d = lane; d < D; d += 32) qs[d] = ldf(qrow + d) * qscale;
-  __syncwarp();
   const int pos = p.ctx_len[b] + t;
   // visible keys: a window that ends at the query, or the query's chunk up to the query
   const int lo = p.chunk > 0 ? (pos / p.chunk) * p.chunk : (p.window > 0 ? max(pos - p.window + 1, 0) : 0);
@@ -284,87 +282,102 @@ __global__ void __launch_bounds__(SPLIT ? 1024 : ATT_WARPS * 32) paged_window_at
   const float slope = p.slopes ? p.slopes[h] : 0.f;
   const int* table = p.block_table + (long long)b * p.max_blocks;
   const bool kvec = ((D * (int)sizeof(T)) % 16) == 0;
-  const T* kc = (const T*)p.k_cache;
   const T* vc = (const T*)p.v_cache;
-  float m = -INFINITY, l = 0.f, acc[ATT_VPL];
-#pragma unroll
-  for (int i = 0; i < ATT_VPL; ++i) acc[i] = 0.f;
   // value rows whose byte size is 16 * 2^k (k <= 5) are read as 16-byte pieces, LPR lanes per row
   constexpr int VN = Vec<T>::N;
   const int LPR = Dv / VN;
   const bool vvec = Dv % VN == 0 && LPR >= 1 && LPR <= 32 && (LPR & (LPR - 1)) == 0 && (p.v_rs * (long long)sizeof(T)) % 16 == 0;
   const int sub = vvec ? lane / LPR : 0, piece = vvec ? lane % LPR : 0;
-  float accv[VN];
-#pragma unroll
-  for (int e = 0; e < VN; ++e) accv[e] = 0.f;
+  const int group = SPLIT ? nwarps / MAPS : 1;                   // warps that share one map's keys
   const int nchunks = (n + 31) / 32;
-  for (int ch = SPLIT ? warp : 0; ch < nchunks; ch += SPLIT ? nwarps : 1) {
-    const int idx = ch * 32 + lane;
-    float s = -INFINITY;
-    long long row = 0;
-    if (idx < n) {
-      const int j = idx < nA ? idx : lo + (idx - nA);
-      row = ((long long)table[j / p.page] * p.page + j % p.page) * p.G + g;
-      s = dot_row(qs, kc + row * D, D, kvec);
-      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
-      s -= slope * (float)(pos - j);
+  float m = -INFINITY, l = 0.f, acc[ATT_VPL], first[MAPS == 2 ? ATT_VPL : 1];
+#pragma unroll 1
+  for (int mi = 0; mi < (SPLIT ? 1 : MAPS); ++mi) {
+    const int map = SPLIT ? warp / group : mi;
+    if (MAPS == 2 && mi == 1) {        // the first map is done: keep its result, start over
+#pragma unroll
+      for (int i = 0; i < ATT_VPL; ++i) first[i] = acc[i] / l;
+      __syncwarp();
     }
-    const float m_new = fmaxf(m, warp_max(s));
-    const float corr = expf(m - m_new);          // m = -inf on the first chunk: exp(-inf) = 0
-    const float pj = idx < n ? expf(s - m_new) : 0.f;
-    l = l * corr + warp_sum(pj);
+    m = -INFINITY;
+    l = 0.f;
 #pragma unroll
-    for (int i = 0; i < ATT_VPL; ++i) acc[i] *= corr;
-    m = m_new;
-    const int cnt = min(32, n - ch * 32);
-    if (vvec) {
-      // LPR lanes read one value row as 16-byte pieces: 32 / LPR keys per load instruction
+    for (int i = 0; i < ATT_VPL; ++i) acc[i] = 0.f;
+    float accv[VN];
 #pragma unroll
-      for (int e = 0; e < VN; ++e) accv[e] *= corr;
-      for (int jj = 0; jj < cnt; jj += 32 / LPR) {
-        const int src = jj + sub;
-        const float pw = __shfl_sync(0xffffffffu, pj, src & 31);
-        const long long r = __shfl_sync(0xffffffffu, row, src & 31);
-        if (src < cnt) {
-          const uint4 raw = *reinterpret_cast<const uint4*>(vc + r * p.v_rs + piece * VN);
-          if constexpr (VN == 4) {
-            accv[0] += pw * __uint_as_float(raw.x); accv[1] += pw * __uint_as_float(raw.y);
-            accv[2] += pw * __uint_as_float(raw.z); accv[3] += pw * __uint_as_float(raw.w);
-          } else {
-            accv[0] += pw * bf16lo(raw.x); accv[1] += pw * bf16hi(raw.x); accv[2] += pw * bf16lo(raw.y); accv[3] += pw * bf16hi(raw.y);
-            accv[4] += pw * bf16lo(raw.z); accv[5] += pw * bf16hi(raw.z); accv[6] += pw * bf16lo(raw.w); accv[7] += pw * bf16hi(raw.w);
+    for (int e = 0; e < VN; ++e) accv[e] = 0.f;
+    const T* qrow = (const T*)p.q + (qi * MAPS + map) * D;
+    for (int d = lane; d < D; d += 32) qs[d] = ldf(qrow + d) * qscale;
+    __syncwarp();
+    const T* kc = (const T*)p.k_cache + (long long)map * D;
+    for (int ch = SPLIT ? warp % group : 0; ch < nchunks; ch += group) {
+      const int idx = ch * 32 + lane;
+      float s = -INFINITY;
+      long long row = 0;
+      if (idx < n) {
+        const int j = idx < nA ? idx : lo + (idx - nA);
+        row = ((long long)table[j / p.page] * p.page + j % p.page) * p.G + g;
+        s = dot_row(qs, kc + row * (MAPS * D), D, kvec);
+        if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+        s -= slope * (float)(pos - j);
+      }
+      const float m_new = fmaxf(m, warp_max(s));
+      const float corr = expf(m - m_new);          // m = -inf on the first chunk: exp(-inf) = 0
+      const float pj = idx < n ? expf(s - m_new) : 0.f;
+      l = l * corr + warp_sum(pj);
+#pragma unroll
+      for (int i = 0; i < ATT_VPL; ++i) acc[i] *= corr;
+      m = m_new;
+      const int cnt = min(32, n - ch * 32);
+      if (vvec) {
+        // LPR lanes read one value row as 16-byte pieces: 32 / LPR keys per load instruction
+#pragma unroll
+        for (int e = 0; e < VN; ++e) accv[e] *= corr;
+        for (int jj = 0; jj < cnt; jj += 32 / LPR) {
+          const int src = jj + sub;
+          const float pw = __shfl_sync(0xffffffffu, pj, src & 31);
+          const long long r = __shfl_sync(0xffffffffu, row, src & 31);
+          if (src < cnt) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(vc + r * p.v_rs + piece * VN);
+            if constexpr (VN == 4) {
+              accv[0] += pw * __uint_as_float(raw.x); accv[1] += pw * __uint_as_float(raw.y);
+              accv[2] += pw * __uint_as_float(raw.z); accv[3] += pw * __uint_as_float(raw.w);
+            } else {
+              accv[0] += pw * bf16lo(raw.x); accv[1] += pw * bf16hi(raw.x); accv[2] += pw * bf16lo(raw.y); accv[3] += pw * bf16hi(raw.y);
+              accv[4] += pw * bf16lo(raw.z); accv[5] += pw * bf16hi(raw.z); accv[6] += pw * bf16lo(raw.w); accv[7] += pw * bf16hi(raw.w);
+            }
+          }
+        }
+      } else {
+        for (int jj = 0; jj < cnt; ++jj) {
+          const float pw = __shfl_sync(0xffffffffu, pj, jj);
+          const long long r = __shfl_sync(0xffffffffu, row, jj);
+          const T* vrow = vc + r * p.v_rs;
+#pragma unroll
+          for (int i = 0; i < ATT_VPL; ++i) {
+            const int dv = lane + 32 * i;
+            if (dv < Dv) acc[i] += pw * ldf(vrow + dv);
           }
         }
       }
-    } else {
-      for (int jj = 0; jj < cnt; ++jj) {
-        const float pw = __shfl_sync(0xffffffffu, pj, jj);
-        const long long r = __shfl_sync(0xffffffffu, row, jj);
-        const T* vrow = vc + r * p.v_rs;
+    }
+    if (vvec) {
+      // fold the lanes that shared a piece, then hand the row over in the (lane + 32 i) layout the epilogue uses
+      for (int o = LPR; o < 32; o <<= 1)
 #pragma unroll
-        for (int i = 0; i < ATT_VPL; ++i) {
-          const int dv = lane + 32 * i;
-          if (dv < Dv) acc[i] += pw * ldf(vrow + dv);
-        }
+        for (int e = 0; e < VN; ++e) accv[e] += __shfl_xor_sync(0xffffffffu, accv[e], o);
+      float* mine = smem + nwarps * D + warp * (Dv + 2);
+      if (sub == 0)
+#pragma unroll
+        for (int e = 0; e < VN; ++e) mine[piece * VN + e] = accv[e];
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < ATT_VPL; ++i) {
+        const int dv = lane + 32 * i;
+        acc[i] = dv < Dv ? mine[dv] : 0.f;
       }
+      __syncwarp();
     }
-  }
-  if (vvec) {
-    // fold the lanes that shared a piece, then hand the row over in the (lane + 32 i) layout the epilogue uses
-    for (int o = LPR; o < 32; o <<= 1)
-#pragma unroll
-      for (int e = 0; e < VN; ++e) accv[e] += __shfl_xor_sync(0xffffffffu, accv[e], o);
-    float* mine = smem + nwarps * D + warp * (Dv + 2);
-    if (sub == 0)
-#pragma unroll
-      for (int e = 0; e < VN; ++e) mine[piece * VN + e] = accv[e];
-    __syncwarp();
-#pragma unroll
-    for (int i = 0; i < ATT_VPL; ++i) {
-      const int dv = lane + 32 * i;
-      acc[i] = dv < Dv ? mine[dv] : 0.f;
-    }
-    __syncwarp();
   }
   if (SPLIT) {
     float* part = smem + nwarps * D + warp * (Dv + 2);
@@ -376,26 +389,46 @@ __global__ void __launch_bounds__(SPLIT ? 1024 : ATT_WARPS * 32) paged_window_at
     if (lane == 0) { part[Dv] = m; part[Dv + 1] = l; }
     __syncthreads();
     if (warp != 0) return;
-    float M = -INFINITY;
-    for (int w = 0; w < nwarps; ++w) M = fmaxf(M, smem[nwarps * D + w * (Dv + 2) + Dv]);
-    l = 0.f;
 #pragma unroll
-    for (int i = 0; i < ATT_VPL; ++i) acc[i] = 0.f;
-    for (int w = 0; w < nwarps; ++w) {
-      const float* pw = smem + nwarps * D + w * (Dv + 2);
-      const float f = pw[Dv] == -INFINITY ? 0.f : expf(pw[Dv] - M);
-      l += pw[Dv + 1] * f;
+    for (int map = 0; map < MAPS; ++map) {
+      if (MAPS == 2 && map == 1)
 #pragma unroll
-      for (int i = 0; i < ATT_VPL; ++i) {
-        const int dv = lane + 32 * i;
-        if (dv < Dv) acc[i] += pw[dv] * f;
+        for (int i = 0; i < ATT_VPL; ++i) first[i] = acc[i] / l;
+      const float* parts = smem + nwarps * D + map * group * (Dv + 2);
+      m = -INFINITY;
+      for (int w = 0; w < group; ++w) m = fmaxf(m, parts[w * (Dv + 2) + Dv]);
+      l = 0.f;
+#pragma unroll
+      for (int i = 0; i < ATT_VPL; ++i) acc[i] = 0.f;
+      for (int w = 0; w < group; ++w) {
+        const float* pw = parts + w * (Dv + 2);
+        const float f = pw[Dv] == -INFINITY ? 0.f : expf(pw[Dv] - m);
+        l += pw[Dv + 1] * f;
+#pragma unroll
+        for (int i = 0; i < ATT_VPL; ++i) {
+          const int dv = lane + 32 * i;
+          if (dv < Dv) acc[i] += pw[dv] * f;
+        }
       }
     }
-    m = M;
+  }
+  T* orow = (T*)p.out + qi * Dv;
+  if constexpr (MAPS == 2) {
+    const float lam = p.lam[0];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < ATT_VPL; ++i) {
+      acc[i] = lane + 32 * i < Dv ? first[i] - lam * (acc[i] / l) : 0.f;
+      ss += acc[i] * acc[i];
+    }
+    const float r = p.diff_scale / sqrtf(warp_sum(ss) / (float)Dv + p.diff_eps);
+#pragma unroll
+    for (int i = 0; i < ATT_VPL; ++i)
+      if (lane + 32 * i < Dv) stf(orow + lane + 32 * i, acc[i] * r);
+    return;
   }
   if (p.sinks) l += expf(p.sinks[h] - m);      // the sink: one more term of the denominator, no value (a live query sees itself: m is finite)
   const float inv = 1.f / l;
-  T* orow = (T*)p.out + qi * Dv;
   const T* grow = p.gate ? (const T*)p.gate + (long long)b * p.g_sb + (long long)t * p.g_st + (p.gate_per_head ? (long long)h : (long long)h * Dv)
                          : nullptr;
   const float head_gate = (grow && p.gate_per_head) ? sigmoidf_acc(ldf(grow)) : 1.f;
@@ -420,35 +453,38 @@ constexpr int MMA_MT = 64, MMA_KT = 64;
 __device__ __forceinline__ float tanh_fast(float x) { return 1.f - __fdividef(2.f, __expf(2.f * x) + 1.f); }
 
 // VPREFIX: the value of a key is the first DV channels of its key row (latent caches): the key tile in shared memory serves both products.
-template <int D, int DV, bool VPREFIX>
-__global__ void __launch_bounds__(128, (D + DV <= 256) ? 3 : 2) paged_window_attention_mma_kernel(WindowAttnParams p) {
-  constexpr int KS = D + 8, VS = VPREFIX ? KS : DV + 8, STAGE = MMA_KT * (VPREFIX ? KS : KS + VS);
+// MAPS = 2 (differential attention): 32 queries per block; warps 0, 1 attend with map 1 and warps 2, 3 with map 2 of the same queries over ONE
+// value tile; at the end the second pair hands its rows to the first through shared memory for the difference, the norm and the scale.
+template <int D, int DV, bool VPREFIX, int MAPS = 1>
+__global__ void __launch_bounds__(128, (D * MAPS + DV <= 256) ? 3 : 2) paged_window_attention_mma_kernel(WindowAttnParams p) {
+  constexpr int KW = D * MAPS, MT = MMA_MT / MAPS;                // key channels per token, queries per block
+  constexpr int KS = KW + 8, VS = VPREFIX ? KS : DV + 8, STAGE = MMA_KT * (VPREFIX ? KS : KS + VS);
   extern __shared__ __align__(16) unsigned char mma_smem[];       // two stages of [64][KS] keys + [64][VS] values
   __nv_bfloat16* stage0 = reinterpret_cast<__nv_bfloat16*>(mma_smem);
-  const int h = blockIdx.y, b = blockIdx.z, t0 = blockIdx.x * MMA_MT;
+  const int h = blockIdx.y, b = blockIdx.z, t0 = blockIdx.x * MT;
   const int qn = p.q_len[b];
   if (t0 >= qn) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+  const int warp = (threadIdx.x >> 5) % (4 / MAPS), map = (threadIdx.x >> 5) / (4 / MAPS), lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
   const int g = h / (p.Hq / p.G), ctx = p.ctx_len[b];
   const int r0 = t0 + warp * 16 + gid, r1 = r0 + 8;            // this thread's two query rows (token index in the row of the batch)
   const int pos0 = ctx + r0, pos1 = ctx + r1;
   uint32_t qa[D / 16][4];
   {
-    const __nv_bfloat16* qb = (const __nv_bfloat16*)p.q + ((long long)b * p.T * p.Hq + h) * D;
+    const __nv_bfloat16* qb = (const __nv_bfloat16*)p.q + ((long long)b * p.T * p.Hq + h) * KW + map * D;
 #pragma unroll
     for (int ks = 0; ks < D / 16; ++ks) {
       const int col = ks * 16 + tig * 2;
-      qa[ks][0] = r0 < p.T ? *reinterpret_cast<const uint32_t*>(qb + (long long)r0 * p.Hq * D + col) : 0u;
-      qa[ks][1] = r1 < p.T ? *reinterpret_cast<const uint32_t*>(qb + (long long)r1 * p.Hq * D + col) : 0u;
-      qa[ks][2] = r0 < p.T ? *reinterpret_cast<const uint32_t*>(qb + (long long)r0 * p.Hq * D + col + 8) : 0u;
-      qa[ks][3] = r1 < p.T ? *reinterpret_cast<const uint32_t*>(qb + (long long)r1 * p.Hq * D + col + 8) : 0u;
+      qa[ks][0] = r0 < p.T ? *reinterpret_cast<const uint32_t*>(qb + (long long)r0 * p.Hq * KW + col) : 0u;
+      qa[ks][1] = r1 < p.T ? *reinterpret_cast<const uint32_t*>(qb + (long long)r1 * p.Hq * KW + col) : 0u;
+      qa[ks][2] = r0 < p.T ? *reinterpret_cast<const uint32_t*>(qb + (long long)r0 * p.Hq * KW + col + 8) : 0u;
+      qa[ks][3] = r1 < p.T ? *reinterpret_cast<const uint32_t*>(qb + (long long)r1 * p.Hq * KW + col + 8) : 0u;
     }
   }
   float o[DV / 8][4];
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-  const int p_first = ctx + t0, p_last = ctx + min(t0 + MMA_MT, qn) - 1;
+  const int p_first = ctx + t0, p_last = ctx + min(t0 + MT, qn) - 1;
   const int lo = p.chunk > 0 ? (p_first / p.chunk) * p.chunk : (p.window > 0 ? max(p_first - p.window + 1, 0) : 0);
   const int nA = p.window > 0 ? min(p.keep_first, lo) : 0;
   const float slope = p.slopes ? p.slopes[h] : 0.f;
@@ -485,7 +521,7 @@ __global__ void __launch_bounds__(128, (D + DV <= 256) ? 3 : 2) paged_window_att
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(cache + row * rs + ch * 8), "r"(nbytes));
       }
     };
-    copy_rows(kc, (long long)D, Kd, std::integral_constant<int, D>{}, std::integral_constant<int, KS>{});
+    copy_rows(kc, (long long)KW, Kd, std::integral_constant<int, KW>{}, std::integral_constant<int, KS>{});
     if constexpr (!VPREFIX) copy_rows(vc, p.v_rs, Vd, std::integral_constant<int, DV>{}, std::integral_constant<int, VS>{});
     asm volatile("cp.async.commit_group;");
   };
@@ -510,7 +546,7 @@ __global__ void __launch_bounds__(128, (D + DV <= 256) ? 3 : 2) paged_window_att
       for (int ks = 0; ks < D / 16; ++ks)
 #pragma unroll
         for (int nt = 0; nt < MMA_KT / 8; ++nt) {
-          const __nv_bfloat16* kp = Ks + (nt * 8 + gid) * KS + ks * 16 + tig * 2;
+          const __nv_bfloat16* kp = Ks + (nt * 8 + gid) * KS + map * D + ks * 16 + tig * 2;
           const uint32_t bb[2] = {*reinterpret_cast<const uint32_t*>(kp), *reinterpret_cast<const uint32_t*>(kp + 8)};
           mma_bf16_16816(sc[nt], qa[ks], bb);
         }
@@ -585,6 +621,36 @@ __global__ void __launch_bounds__(128, (D + DV <= 256) ? 3 : 2) paged_window_att
     l1 += __expf(sk - m1);
   }
   float i0 = 1.f / l0, i1 = 1.f / l1;
+  if constexpr (MAPS == 2) {
+    constexpr int OS = DV + 2;
+    float* second = reinterpret_cast<float*>(mma_smem);           // [MT][OS]; the key / value stages are done with (barrier after the last tile)
+    const int lr0 = warp * 16 + gid, lr1 = lr0 + 8;
+    if (map == 1) {
+#pragma unroll
+      for (int nv = 0; nv < DV / 8; ++nv) {
+        const int col = nv * 8 + tig * 2;
+        *reinterpret_cast<float2*>(second + lr0 * OS + col) = make_float2(o[nv][0] * i0, o[nv][1] * i0);
+        *reinterpret_cast<float2*>(second + lr1 * OS + col) = make_float2(o[nv][2] * i1, o[nv][3] * i1);
+      }
+    }
+    __syncthreads();
+    if (map == 1) return;
+    const float lam = p.lam[0];
+    float q0 = 0.f, q1 = 0.f;
+#pragma unroll
+    for (int nv = 0; nv < DV / 8; ++nv) {
+      const int col = nv * 8 + tig * 2;
+      const float2 b0 = *reinterpret_cast<const float2*>(second + lr0 * OS + col), b1 = *reinterpret_cast<const float2*>(second + lr1 * OS + col);
+      o[nv][0] = o[nv][0] * i0 - lam * b0.x; o[nv][1] = o[nv][1] * i0 - lam * b0.y;
+      o[nv][2] = o[nv][2] * i1 - lam * b1.x; o[nv][3] = o[nv][3] * i1 - lam * b1.y;
+      q0 += o[nv][0] * o[nv][0] + o[nv][1] * o[nv][1];
+      q1 += o[nv][2] * o[nv][2] + o[nv][3] * o[nv][3];
+    }
+    q0 += __shfl_xor_sync(0xffffffffu, q0, 1); q0 += __shfl_xor_sync(0xffffffffu, q0, 2);
+    q1 += __shfl_xor_sync(0xffffffffu, q1, 1); q1 += __shfl_xor_sync(0xffffffffu, q1, 2);
+    i0 = p.diff_scale / sqrtf(q0 / (float)DV + p.diff_eps);
+    i1 = p.diff_scale / sqrtf(q1 / (float)DV + p.diff_eps);
+  }
   __nv_bfloat16* ob = (__nv_bfloat16*)p.out + ((long long)b * p.T * p.Hq + h) * DV;
   const __nv_bfloat16* gb = (p.gate && !p.gate_per_head) ? (const __nv_bfloat16*)p.gate + (long long)b * p.g_sb + (long long)h * DV : nullptr;
   if (p.gate && p.gate_per_head) {
@@ -740,9 +806,11 @@ __global__ void __launch_bounds__(SCAN_THREADS, NB == 1 ? 4 : 2) ssd_scan_kernel
 }
 
 // ---- grouped RMS norm ---------------------------------------------------------------------------------------------------------
+__device__ __forceinline__ float unary_apply(int act, float v);
 template <typename TO>
 __global__ void __launch_bounds__(256) group_rmsnorm_kernel(const float* __restrict__ y, const float* __restrict__ w, TO* __restrict__ out,
-                                                            int W, int gw, float eps) {
+                                                            int W, int gw, float eps, const void* __restrict__ gate, long long g_stride, int g_lp,
+                                                            int act) {
   __shared__ float red[32];
   const long long base = (long long)blockIdx.x * W + (long long)blockIdx.y * gw;      // rows on grid.x: no 65535 limit
   float ss = 0.f;
@@ -752,7 +820,12 @@ __global__ void __launch_bounds__(256) group_rmsnorm_kernel(const float* __restr
   }
   ss = block_sum(ss, red);
   const float r = 1.f / sqrtf(ss / (float)gw + eps);
-  for (int c = threadIdx.x; c < gw; c += blockDim.x) stf(out + base + c, y[base + c] * r * w[blockIdx.y * gw + c]);
+  const long long gb = (long long)blockIdx.x * g_stride + (long long)blockIdx.y * gw;
+  for (int c = threadIdx.x; c < gw; c += blockDim.x) {
+    float v = y[base + c] * r * w[blockIdx.y * gw + c];
+    if (gate) v *= unary_apply(act, g_lp ? __bfloat162float(((const __nv_bfloat16*)gate)[gb + c]) : ((const float*)gate)[gb + c]);
+    stf(out + base + c, v);
+  }
 }
 
 // ---- clamped gate product -----------------------------------------------------------------------------------------------------
@@ -1570,8 +1643,8 @@ __global__ void __launch_bounds__(HNR_WARPS * 32) head_norm_rope_append_kernel(H
   }
   if (!p.value_from_key) {
     const T* vs = row + Cq + Ck;
-    T* vo = (T*)p.v_cache + slot * p.n_kv * Dv;
-    for (int c = threadIdx.x; c < p.n_kv * Dv; c += blockDim.x) vo[c] = vs[c];
+    T* vo = (T*)p.v_cache + slot * p.n_v * Dv;
+    for (int c = threadIdx.x; c < p.n_v * Dv; c += blockDim.x) vo[c] = vs[c];
   }
 }
 
@@ -1663,9 +1736,9 @@ __global__ void __launch_bounds__(HNR_WARPS * 32) head_norm_rope_append_lane_ker
   }
   if (!p.value_from_key) {
     const T* vs = row + Cq + Ck;
-    T* vo = (T*)p.v_cache + slot * p.n_kv * Dv;
+    T* vo = (T*)p.v_cache + slot * p.n_v * Dv;
     constexpr int VN = Vec<T>::N;
-    const int n = p.n_kv * Dv;
+    const int n = p.n_v * Dv;
     if (n % VN == 0 && (((uintptr_t)vs | (uintptr_t)vo) & 15) == 0) {
       for (int c = threadIdx.x * VN; c < n; c += blockDim.x * VN) *reinterpret_cast<uint4*>(vo + c) = *reinterpret_cast<const uint4*>(vs + c);
     } else {
@@ -2226,9 +2299,9 @@ void paged_window_attention_launch(const WindowAttnParams& p, bool lp, cudaStrea
   const long long nq = (long long)p.B * p.T * p.Hq;
   if (nq <= 0) return;
   // values that are a prefix of the key rows of the same cache (latent rows with a rotated tail): one shared-memory tile serves both
-  const bool prefix = p.v_cache == p.k_cache && p.v_rs == p.D && p.G == 1;
+  const bool prefix = p.maps != 2 && p.v_cache == p.k_cache && p.v_rs == p.D && p.G == 1;
   const bool rows16 = (p.v_rs * 2) % 16 == 0;
-  if (lp && p.T >= 16 && rows16 && ((!prefix && (p.D == 64 || p.D == 128) && (p.Dv == 64 || p.Dv == 128)) ||
+  if (lp && p.maps != 2 && p.T >= 16 && rows16 && ((!prefix && (p.D == 64 || p.D == 128) && (p.Dv == 64 || p.Dv == 128)) ||
                                     (prefix && ((p.D == 80 && p.Dv == 64) || (p.D == 192 && p.Dv == 128) || (p.D == p.Dv && (p.D == 64 || p.D == 128)))))) {
     // prompt portions in bf16: tensor-core kernel
     dim3 grid((p.T + MMA_MT - 1) / MMA_MT, p.Hq, p.B);
@@ -2248,24 +2321,43 @@ void paged_window_attention_launch(const WindowAttnParams& p, bool lp, cudaStrea
     else go(paged_window_attention_mma_kernel<128, 128, false>);
     return;
   }
+  const bool two = p.maps == 2;
+  if (two && lp && p.T >= 16 && rows16 && (p.D == 64 || p.D == 128) && (p.Dv == 64 || p.Dv == 128)) {
+    dim3 grid((p.T + MMA_MT / 2 - 1) / (MMA_MT / 2), p.Hq, p.B);
+    const size_t smem = 2 * (size_t)MMA_KT * (2 * p.D + 8 + p.Dv + 8) * sizeof(__nv_bfloat16);
+    auto go = [&](auto kernel) {
+      opt_in_smem(kernel, smem);
+      kernel<<<grid, 128, smem, st>>>(p);
+    };
+    if (p.D == 64 && p.Dv == 64) go(paged_window_attention_mma_kernel<64, 64, false, 2>);
+    else if (p.D == 64) go(paged_window_attention_mma_kernel<64, 128, false, 2>);
+    else if (p.Dv == 64) go(paged_window_attention_mma_kernel<128, 64, false, 2>);
+    else go(paged_window_attention_mma_kernel<128, 128, false, 2>);
+    return;
+  }
   // few queries (decode steps): one block per query, its warps split the keys; otherwise one warp per query
   const bool split = nq <= 2LL * kNumSMs * 4;
   // split mode: one warp per 32 visible keys (bounded by the window or by the pages a row can hold), 4 to 32 warps
   long long span = (long long)p.max_blocks * p.page;
   if (p.window > 0) span = std::min<long long>(span, (long long)p.window + p.keep_first);
   if (p.chunk > 0) span = std::min<long long>(span, (long long)p.chunk);
-  const int nwarps = split ? (int)std::min<long long>(32, std::max<long long>(ATT_WARPS, (span + 31) / 32)) : ATT_WARPS;
+  const int maps = two ? 2 : 1;          // two maps: half of the warps each
+  const int nwarps = split ? maps * (int)std::min<long long>(32 / maps, std::max<long long>(ATT_WARPS, (span + 31) / 32)) : ATT_WARPS;
   const size_t smem = sizeof(float) * (size_t)(nwarps * (p.D + p.Dv + 2));
   const unsigned grid = (unsigned)(split ? nq : (nq + ATT_WARPS - 1) / ATT_WARPS);
   auto go = [&](auto kernel) {
     opt_in_smem(kernel, smem);
     kernel<<<grid, nwarps * 32, smem, st>>>(p);
   };
-  if (lp) {
-    if (split) go(paged_window_attention_kernel<__nv_bfloat16, true>); else go(paged_window_attention_kernel<__nv_bfloat16, false>);
-  } else {
-    if (split) go(paged_window_attention_kernel<float, true>); else go(paged_window_attention_kernel<float, false>);
-  }
+  auto pick = [&](auto tag) {
+    using T = decltype(tag);
+    if (two) {
+      if (split) go(paged_window_attention_kernel<T, true, 2>); else go(paged_window_attention_kernel<T, false, 2>);
+    } else {
+      if (split) go(paged_window_attention_kernel<T, true, 1>); else go(paged_window_attention_kernel<T, false, 1>);
+    }
+  };
+  if (lp) pick(__nv_bfloat16{}); else pick(float{});
 }
 
 void ssd_scan_launch(const SsdScanParams& p, bool lp, cudaStream_t st) {
@@ -2383,13 +2475,14 @@ void head_rmsnorm_gate_launch(const float* y, const float* w, const void* gate, 
   }
 }
 
-void group_rmsnorm_launch(const float* y, const float* w, void* out, bool out_lp, int rows, int W, int groups, float eps, cudaStream_t st) {
+void group_rmsnorm_launch(const float* y, const float* w, void* out, bool out_lp, int rows, int W, int groups, float eps, const void* gate,
+                          long long g_stride, bool gate_lp, int act, cudaStream_t st) {
   if (rows <= 0) return;
   dim3 grid(rows, groups);
   if (out_lp)
-    group_rmsnorm_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(y, w, (__nv_bfloat16*)out, W, W / groups, eps);
+    group_rmsnorm_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(y, w, (__nv_bfloat16*)out, W, W / groups, eps, gate, g_stride, (int)gate_lp, act);
   else
-    group_rmsnorm_kernel<float><<<grid, 256, 0, st>>>(y, w, (float*)out, W, W / groups, eps);
+    group_rmsnorm_kernel<float><<<grid, 256, 0, st>>>(y, w, (float*)out, W, W / groups, eps, gate, g_stride, (int)gate_lp, act);
 }
 
 void clamped_glu_launch(const void* gu, void* out, long long rows, int F, float limit, float alpha, bool lp, cudaStream_t st) {

@@ -10,6 +10,7 @@ namespace nxdi {
 constexpr int SEQMIX_MAX_TAPS = 8;       // short convolutions: taps per channel
 constexpr int SEQMIX_MAX_VDIM = 256;     // attention: value channels per head
 constexpr int SEQMIX_MAX_STATE = 256;    // scan: state size per head
+constexpr int SEQMIX_MAX_STREAMS = 8;    // residual streams per token
 
 void scaled_add_rmsnorm_launch(const float* x, const void* y, bool y_lp, const float* w, float* out, void* out_lp, int rows, int W,
                                float alpha, float eps, float offset, cudaStream_t st);
@@ -75,9 +76,11 @@ void moe_plain_gemm_launch(const void* a, const void* w, void* c, int R, int N, 
 void moe_plain_combine_launch(const void* y, const float* topk_w, const int* pos, void* out, int N, int H, int k, bool lp, cudaStream_t st);
 // gated: w_up holds [gate; up] rows ([E, 2 I, H]) and the hidden row is act(gate . x) * (up . x)
 void moe_plain_decode_launch(const void* x, const void* w_up, const void* w_down, const float* topk_w, const int* topk_i, void* h, void* out,
-                             int N, int k, int H, int I, int expert_offset, int e_local, int act, bool gated, bool lp, cudaStream_t st);
+                             int N, int k, int H, int I, int expert_offset, int e_local, int act, bool gated, float limit, float alpha, bool lp,
+                             cudaStream_t st);      // act 7 (gated only): clamped, shifted gate product with limit and alpha
 // h[r, i] = act(gu[r, i]) * gu[r, I + i] for the rows of used 128-row tiles
-void moe_plain_gate_mul_launch(const void* gu, void* h, int R, int I, int act, const int* tile_expert, bool lp, cudaStream_t st);
+void moe_plain_gate_mul_launch(const void* gu, void* h, int R, int I, int act, float limit, float alpha, const int* tile_expert, bool lp,
+                               cudaStream_t st);
 
 // fp32 router: logits = x W^T (x bf16 or fp32, W fp32 [E, W]) on CUDA cores with the rows in shared memory, then per token the
 // scores (sigmoid, or softmax over all E) of the k experts with the largest score + correction among the `keep` best of `groups` equal
@@ -128,6 +131,11 @@ struct WindowAttnParams {
   int chunk;                // > 0: key j is visible from position p only when j / chunk == p / chunk (instead of a window)
   const float* slopes;      // [Hq] or null: slopes[h] * (p - j) is taken off the score of head h
   const float* head_scale;  // [Hq] or null: the score of head h is multiplied by head_scale[h] as well (a learned temperature per head)
+  // differential attention (maps = 2): q [B, T, 2 Hq, D] and the key rows [.., 2 G, D] hold (map 1, map 2) per head, the values [.., G, Dv] serve
+  // both; the output of a head is (a1 - lam[0] a2) divided by its root mean square over Dv (+ diff_eps), times diff_scale
+  int maps;                 // 1 (or 0), 2
+  const float* lam;
+  float diff_scale, diff_eps;
   long long v_rs;           // elements between the value rows of neighbouring (token, kv head) pairs; Dv <= v_rs (values that are a
                             // prefix of a wider cache row: v_cache = k_cache, v_rs = D)
 };
@@ -172,7 +180,7 @@ struct HeadNormRopeParams {
   void* q_out;              // [B, T, n_q, D]
   void *k_cache, *v_cache;  // [blocks, page, n_kv, D | Dv]
   const int *block_table, *ctx_len, *q_len;
-  int B, T, n_q, n_kv, D, Dv, R, page, max_blocks;
+  int B, T, n_q, n_kv, n_v, D, Dv, R, page, max_blocks;      // n_v: value heads
   int norm_at;              // 0 none, 1 before the rotation, 2 after it
   int value_from_key;
   float eps;
@@ -198,8 +206,63 @@ void gated_delta_scan_launch(const DeltaScanParams& p, bool lp, cudaStream_t st)
 void head_rmsnorm_gate_launch(const float* y, const float* w, const void* gate, long long g_stride, void* out, long long rows, int H, int Dv,
                               float eps, int act, bool gate_lp, bool out_lp, cudaStream_t st);
 
-void group_rmsnorm_launch(const float* y, const float* w, void* out, bool out_lp, int rows, int W, int groups, float eps, cudaStream_t st);
+// gate non-null: times act(gate) after the norm; gate rows g_stride elements apart
+void group_rmsnorm_launch(const float* y, const float* w, void* out, bool out_lp, int rows, int W, int groups, float eps, const void* gate,
+                          long long g_stride, bool gate_lp, int act, cudaStream_t st);
 
 void clamped_glu_launch(const void* gu, void* out, long long rows, int F, float limit, float alpha, bool lp, cudaStream_t st);
+
+// Several fp32 residual streams (stream_mix.cu): x'_t = sum_s mix[s, t] x_s + out[t] y; u = sum_s in[s] x'_s; h = rms_unit(u) * w;
+// r_p = h_p + sum_j cw[:, j] h_(p - K + 1 + j) with the K - 1 rows before a portion from the state line, which is advanced.
+struct StreamMixParams {
+  const float* x;                  // streams of token i: x + i * x_tok + s * x_str (x_str = 0: all streams equal)
+  long long x_tok, x_str;
+  const void* y;                   // [B, T, W] bf16 or fp32, or null (no write-back: x' = x)
+  int y_lp;
+  const float *mix, *out_w, *in_w; // [S, S] (from, to), [S], [S]
+  const float* norm_w;
+  int norm_n;                      // 0: no norm, 1: one number, W: a vector
+  const float* conv_w;             // [W, K] or null
+  float* state;                    // [lines, K - 1, W] or null (K == 1)
+  const int *lines, *ctx_len, *q_len;      // q_len null: every row is live; lines / ctx_len are read with a state only
+  float* xn;                       // [B, T, S, W] or null
+  void* h;                         // [B, T, W] bf16 or fp32
+  int B, T, S, W, K;
+  float eps;
+};
+void stream_mix_norm_conv_launch(const StreamMixParams& p, bool h_lp, cudaStream_t st);
+
+// Rows of a gated delta rule with per-channel decays (linear_scan.cu): q | k | v through a short causal convolution (carried rows advanced)
+// and SiLU, unit-length q (times D^-1/2) and k per head; decay = exp(-exp(A_log) softplus(a + dt_bias)); beta = sigmoid(b).
+struct DeltaFrontParams {
+  const void* p;                   // [B, T, >= 2 n_qk D + nh Dv], row strides below
+  long long p_sb, p_st;
+  const void *b_raw, *a_raw;       // [B, T, nh] and [B, T, nh D] views
+  long long b_sb, b_st, a_sb, a_st;
+  const float *conv_w, *A_log, *dt_bias;
+  void* state;                     // [lines, K - 1, 2 n_qk D + nh Dv] of the activation type
+  const int *lines, *ctx_len, *q_len;
+  float *qkv, *decay, *beta;       // [B, T, C], [B, T, nh D], [B, T, nh]
+  int B, T, K, nh, n_qk, D, Dv;
+  float unit_eps;
+};
+void delta_front_launch(const DeltaFrontParams& p, bool lp, cudaStream_t st);
+
+// Recurrences over a state [lines, nh, Dv, D] (value channel by key channel).  delta: rows shrink by decay [B, T, nh D] per key channel, are
+// corrected along k towards v with strength beta, and read after the correction.  Otherwise: M = decay[h] M + outer(k, v), y = M' q.
+struct LinearScanParams {
+  const void* x;                   // rows q | k | v, strides below; fp32 for delta, activation type otherwise
+  long long x_sb, x_st;
+  const float *decay, *beta;       // delta: [B, T, nh D], [B, T, nh]; otherwise decay [nh]
+  float* state;
+  const int *lines, *ctx_len, *q_len;
+  float* y;                        // [B, T, nh Dv]
+  int B, T, nh, n_qk, D, Dv, silu; // silu: SiLU on q, k and v as they are read (fixed decays only)
+};
+void channel_delta_scan_launch(const LinearScanParams& p, cudaStream_t st);
+void decay_scan_launch(const LinearScanParams& p, bool lp, cudaStream_t st);
+
+// idx[i, j] = table[ids[i], j] (-1 for tokens past q_len), w[i, j] = 1 / k
+void table_route_launch(const int* table, const int* ids, const int* q_len, float* w, int* idx, int B, int T, int k, int vocab, cudaStream_t st);
 
 }  // namespace nxdi

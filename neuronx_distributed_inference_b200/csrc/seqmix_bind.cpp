@@ -236,13 +236,191 @@ at::Tensor ssd_scan(const at::Tensor& xBC, const at::Tensor& dt_raw, const at::T
   return y;
 }
 
-at::Tensor group_rmsnorm(const at::Tensor& y, const at::Tensor& w, int64_t groups, double eps, bool out_lp) {
+std::tuple<OptT, at::Tensor> stream_mix_norm_conv(const at::Tensor& x, const OptT& y, const OptT& mix, const OptT& out_w, const at::Tensor& in_w,
+                                                  const OptT& norm_w, const OptT& conv_w, const OptT& state, const OptT& lines, const OptT& ctx,
+                                                  const OptT& qlen, double eps, bool h_lp) {
+  check_f32(x, "stream_mix_norm_conv x");
+  check_f32(in_w, "stream_mix_norm_conv in");
+  const int64_t S = in_w.numel();
+  TORCH_CHECK((x.dim() == 3 || (x.dim() == 4 && x.size(2) == S)) && S >= 1 && S <= SEQMIX_MAX_STREAMS, "stream_mix_norm_conv: x [B, T, W] or [B, T, S, W], S <= ",
+              SEQMIX_MAX_STREAMS);
+  const int64_t B = x.size(0), T = x.size(1), W = x.size(x.dim() - 1);
+  StreamMixParams p{};
+  p.x = x.data_ptr<float>();
+  p.x_tok = x.stride(1);
+  p.x_str = x.dim() == 4 ? W : 0;
+  c10::cuda::CUDAGuard guard(x.device());
+  OptT xn;
+  if (y.has_value()) {
+    check_act(*y, "stream_mix_norm_conv y");
+    TORCH_CHECK(y->is_contiguous() && y->numel() == B * T * W && mix.has_value() && out_w.has_value(), "stream_mix_norm_conv: y [B, T, W] with mix and out");
+    check_f32(*mix, "mix");
+    check_f32(*out_w, "out");
+    TORCH_CHECK(mix->numel() == S * S && out_w->numel() == S);
+    xn = at::empty({B, T, S, W}, x.options());
+    p.y = y->data_ptr(); p.y_lp = is_lp(*y) ? 1 : 0;
+    p.mix = mix->data_ptr<float>(); p.out_w = out_w->data_ptr<float>(); p.xn = xn->data_ptr<float>();
+  }
+  p.in_w = in_w.data_ptr<float>();
+  if (norm_w.has_value()) {
+    check_f32(*norm_w, "norm weight");
+    TORCH_CHECK(norm_w->numel() == 1 || norm_w->numel() == W, "norm weight: one number or one per channel");
+    p.norm_w = norm_w->data_ptr<float>(); p.norm_n = (int)norm_w->numel();
+  }
+  p.K = 1;
+  if (conv_w.has_value()) {
+    check_f32(*conv_w, "convolution weight");
+    TORCH_CHECK(conv_w->dim() == 2 && conv_w->size(0) == W && conv_w->size(1) >= 1 && conv_w->size(1) <= SEQMIX_MAX_TAPS, "convolution weight [W, taps], taps <= ",
+                SEQMIX_MAX_TAPS);
+    p.conv_w = conv_w->data_ptr<float>(); p.K = (int)conv_w->size(1);
+    if (p.K > 1) {
+      TORCH_CHECK(state.has_value() && lines.has_value() && ctx.has_value() && qlen.has_value(), "stream_mix_norm_conv: carried rows need state, lines, ctx_len, q_len");
+      check_f32(*state, "state");
+      TORCH_CHECK(state->dim() == 3 && state->size(1) == p.K - 1 && state->size(2) == W, "state [lines, taps - 1, W]");
+      p.state = state->data_ptr<float>();
+    }
+  }
+  if (lines.has_value()) { check_i32(*lines, B, "lines"); p.lines = lines->data_ptr<int>(); }
+  if (ctx.has_value()) { check_i32(*ctx, B, "ctx_len"); p.ctx_len = ctx->data_ptr<int>(); }
+  if (qlen.has_value()) { check_i32(*qlen, B, "q_len"); p.q_len = qlen->data_ptr<int>(); }
+  auto h = at::empty({B, T, W}, x.options().dtype(h_lp ? at::kBFloat16 : at::kFloat));
+  p.h = h.data_ptr();
+  p.B = (int)B; p.T = (int)T; p.S = (int)S; p.W = (int)W; p.eps = (float)eps;
+  stream_mix_norm_conv_launch(p, h_lp, stream());
+  return {xn, h};
+}
+
+at::Tensor paged_diff_attention(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, const at::Tensor& block_table,
+                                const at::Tensor& ctx, const at::Tensor& qlen, double scale, const at::Tensor& lam, double out_scale, double eps,
+                                int64_t window) {
+  check_act(q, "paged_diff_attention q");
+  TORCH_CHECK(q.dim() == 4 && q.is_contiguous() && q.size(2) % 2 == 0, "paged_diff_attention: q [B, T, 2 heads, D]");
+  const int64_t B = q.size(0), T = q.size(1), H = q.size(2) / 2, D = q.size(3);
+  TORCH_CHECK(k_cache.is_cuda() && k_cache.scalar_type() == q.scalar_type() && k_cache.is_contiguous() && k_cache.dim() == 4 && k_cache.size(3) == D &&
+              k_cache.size(2) % 2 == 0, "paged_diff_attention: key cache [blocks, page, 2 kv heads, D]");
+  const int64_t G = k_cache.size(2) / 2;
+  TORCH_CHECK(v_cache.is_cuda() && v_cache.scalar_type() == q.scalar_type() && v_cache.is_contiguous() && v_cache.dim() == 4 && v_cache.size(0) == k_cache.size(0) &&
+              v_cache.size(1) == k_cache.size(1) && v_cache.size(2) == G, "paged_diff_attention: value cache [blocks, page, kv heads, Dv]");
+  const int64_t Dv = v_cache.size(3);
+  TORCH_CHECK(H % G == 0 && Dv <= SEQMIX_MAX_VDIM, "paged_diff_attention: heads must divide, value size <= ", SEQMIX_MAX_VDIM);
+  TORCH_CHECK(block_table.is_cuda() && block_table.scalar_type() == at::kInt && block_table.is_contiguous() && block_table.dim() == 2 &&
+              block_table.size(0) == B);
+  check_i32(ctx, B, "ctx_len");
+  check_i32(qlen, B, "q_len");
+  check_f32(lam, "lambda");
+  TORCH_CHECK(lam.numel() == 1);
+  c10::cuda::CUDAGuard guard(q.device());
+  auto out = at::zeros({B, T, H * Dv}, q.options());
+  WindowAttnParams a{};
+  a.maps = 2; a.lam = lam.data_ptr<float>(); a.diff_scale = (float)out_scale; a.diff_eps = (float)eps;
+  a.q = q.data_ptr(); a.k_cache = k_cache.data_ptr(); a.v_cache = v_cache.data_ptr(); a.v_rs = Dv;
+  a.block_table = block_table.data_ptr<int>(); a.ctx_len = ctx.data_ptr<int>(); a.q_len = qlen.data_ptr<int>();
+  a.out = out.data_ptr();
+  a.B = (int)B; a.T = (int)T; a.Hq = (int)H; a.G = (int)G; a.D = (int)D; a.Dv = (int)Dv; a.page = (int)k_cache.size(1);
+  a.max_blocks = (int)block_table.size(1); a.window = (int)window; a.scale = (float)scale;
+  paged_window_attention_launch(a, is_lp(q), stream());
+  return out;
+}
+
+std::tuple<at::Tensor, at::Tensor, at::Tensor> delta_front(const at::Tensor& pr, const at::Tensor& b_raw, const at::Tensor& a_raw, const at::Tensor& conv_w,
+                                                           const at::Tensor& A_log, const at::Tensor& dt_bias, at::Tensor state, const at::Tensor& lines,
+                                                           const at::Tensor& ctx, const at::Tensor& qlen, int64_t nh, int64_t n_qk, int64_t D, int64_t Dv,
+                                                           double unit_eps) {
+  check_act(pr, "delta_front rows");
+  check_rows(pr, "delta_front rows");
+  const int64_t B = pr.size(0), T = pr.size(1), C = 2 * n_qk * D + nh * Dv, K = conv_w.size(1);
+  TORCH_CHECK(pr.size(2) >= C && nh % n_qk == 0 && D >= 1 && D <= 256, "delta_front: rows q | k | v, key size <= 256");
+  for (const at::Tensor* t : {&b_raw, &a_raw}) {
+    check_rows(*t, "delta_front beta / decay rows");
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == pr.scalar_type() && t->size(0) == B && t->size(1) == T);
+  }
+  TORCH_CHECK(b_raw.size(2) == nh && a_raw.size(2) == nh * D, "delta_front: beta [B, T, heads], decay [B, T, heads * D]");
+  check_f32(conv_w, "conv weight"); check_f32(A_log, "A_log"); check_f32(dt_bias, "dt_bias");
+  TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(0) == C && K >= 1 && K <= SEQMIX_MAX_TAPS && A_log.numel() == nh && dt_bias.numel() == nh * D);
+  TORCH_CHECK(state.is_cuda() && state.scalar_type() == pr.scalar_type() && state.is_contiguous() && state.dim() == 3 && state.size(1) == K - 1 &&
+              state.size(2) == C, "delta_front: state [lines, taps - 1, q | k | v channels] of the activation type");
+  check_i32(lines, B, "lines"); check_i32(ctx, B, "ctx_len"); check_i32(qlen, B, "q_len");
+  c10::cuda::CUDAGuard guard(pr.device());
+  auto f32 = pr.options().dtype(at::kFloat);
+  auto qkv = at::empty({B, T, C}, f32), decay = at::empty({B, T, nh * D}, f32), beta = at::empty({B, T, nh}, f32);
+  DeltaFrontParams p{};
+  p.p = pr.data_ptr(); p.p_sb = pr.stride(0); p.p_st = pr.stride(1);
+  p.b_raw = b_raw.data_ptr(); p.b_sb = b_raw.stride(0); p.b_st = b_raw.stride(1);
+  p.a_raw = a_raw.data_ptr(); p.a_sb = a_raw.stride(0); p.a_st = a_raw.stride(1);
+  p.conv_w = conv_w.data_ptr<float>(); p.A_log = A_log.data_ptr<float>(); p.dt_bias = dt_bias.data_ptr<float>(); p.state = state.data_ptr();
+  p.lines = lines.data_ptr<int>(); p.ctx_len = ctx.data_ptr<int>(); p.q_len = qlen.data_ptr<int>();
+  p.qkv = qkv.data_ptr<float>(); p.decay = decay.data_ptr<float>(); p.beta = beta.data_ptr<float>();
+  p.B = (int)B; p.T = (int)T; p.K = (int)K; p.nh = (int)nh; p.n_qk = (int)n_qk; p.D = (int)D; p.Dv = (int)Dv; p.unit_eps = (float)unit_eps;
+  delta_front_launch(p, is_lp(pr), stream());
+  return {qkv, decay, beta};
+}
+
+at::Tensor channel_delta_scan(const at::Tensor& qkv, const at::Tensor& decay, const at::Tensor& beta, at::Tensor state, const at::Tensor& lines,
+                              const at::Tensor& ctx, const at::Tensor& qlen, int64_t nh, int64_t n_qk, int64_t D, int64_t Dv) {
+  check_f32(qkv, "channel_delta_scan q | k | v"); check_f32(decay, "channel_delta_scan decay"); check_f32(beta, "channel_delta_scan beta");
+  check_f32(state, "channel_delta_scan state");
+  TORCH_CHECK(qkv.dim() == 3 && qkv.size(2) == 2 * n_qk * D + nh * Dv && nh % n_qk == 0 && D >= 1 && D <= 256, "channel_delta_scan: sizes (D <= 256)");
+  const int64_t B = qkv.size(0), T = qkv.size(1);
+  TORCH_CHECK(decay.numel() == B * T * nh * D && beta.numel() == B * T * nh);
+  TORCH_CHECK(state.dim() == 4 && state.size(1) == nh && state.size(2) == Dv && state.size(3) == D, "channel_delta_scan: state [lines, heads, Dv, D]");
+  check_i32(lines, B, "lines"); check_i32(ctx, B, "ctx_len"); check_i32(qlen, B, "q_len");
+  c10::cuda::CUDAGuard guard(qkv.device());
+  auto y = at::zeros({B, T, nh * Dv}, qkv.options());
+  LinearScanParams p{};
+  p.x = qkv.data_ptr(); p.x_sb = qkv.stride(0); p.x_st = qkv.stride(1);
+  p.decay = decay.data_ptr<float>(); p.beta = beta.data_ptr<float>(); p.state = state.data_ptr<float>();
+  p.lines = lines.data_ptr<int>(); p.ctx_len = ctx.data_ptr<int>(); p.q_len = qlen.data_ptr<int>(); p.y = y.data_ptr<float>();
+  p.B = (int)B; p.T = (int)T; p.nh = (int)nh; p.n_qk = (int)n_qk; p.D = (int)D; p.Dv = (int)Dv;
+  channel_delta_scan_launch(p, stream());
+  return y;
+}
+
+at::Tensor decay_scan(const at::Tensor& x, const at::Tensor& decay, at::Tensor state, const at::Tensor& lines, const at::Tensor& ctx,
+                      const at::Tensor& qlen, int64_t nh, int64_t D, int64_t Dv, bool silu) {
+  check_act(x, "decay_scan rows");
+  check_rows(x, "decay_scan rows");
+  check_f32(decay, "decay_scan decay"); check_f32(state, "decay_scan state");
+  const int64_t B = x.size(0), T = x.size(1);
+  TORCH_CHECK(x.size(2) >= nh * (2 * D + Dv) && decay.numel() == nh && D >= 1 && D <= 256, "decay_scan: rows q | k | v, one decay per head, key size <= 256");
+  TORCH_CHECK(state.dim() == 4 && state.size(1) == nh && state.size(2) == Dv && state.size(3) == D, "decay_scan: state [lines, heads, Dv, D]");
+  check_i32(lines, B, "lines"); check_i32(ctx, B, "ctx_len"); check_i32(qlen, B, "q_len");
+  c10::cuda::CUDAGuard guard(x.device());
+  auto y = at::zeros({B, T, nh * Dv}, x.options().dtype(at::kFloat));
+  LinearScanParams p{};
+  p.x = x.data_ptr(); p.x_sb = x.stride(0); p.x_st = x.stride(1);
+  p.decay = decay.data_ptr<float>(); p.state = state.data_ptr<float>();
+  p.lines = lines.data_ptr<int>(); p.ctx_len = ctx.data_ptr<int>(); p.q_len = qlen.data_ptr<int>(); p.y = y.data_ptr<float>();
+  p.B = (int)B; p.T = (int)T; p.nh = p.n_qk = (int)nh; p.D = (int)D; p.Dv = (int)Dv; p.silu = silu ? 1 : 0;
+  decay_scan_launch(p, is_lp(x), stream());
+  return y;
+}
+
+std::tuple<at::Tensor, at::Tensor> table_route(const at::Tensor& table, const at::Tensor& ids, const at::Tensor& qlen) {
+  TORCH_CHECK(table.is_cuda() && table.scalar_type() == at::kInt && table.is_contiguous() && table.dim() == 2, "table_route: table [vocab, k] int32");
+  TORCH_CHECK(ids.dim() == 2);
+  const int64_t B = ids.size(0), T = ids.size(1), k = table.size(1);
+  check_i32(ids, B * T, "token ids");
+  check_i32(qlen, B, "q_len");
+  c10::cuda::CUDAGuard guard(table.device());
+  auto w = at::empty({B * T, k}, table.options().dtype(at::kFloat));
+  auto idx = at::empty({B * T, k}, table.options());
+  table_route_launch(table.data_ptr<int>(), ids.data_ptr<int>(), qlen.data_ptr<int>(), w.data_ptr<float>(), idx.data_ptr<int>(), (int)B, (int)T, (int)k,
+                     (int)table.size(0), stream());
+  return {w, idx};
+}
+
+at::Tensor group_rmsnorm(const at::Tensor& y, const at::Tensor& w, int64_t groups, double eps, bool out_lp, const OptT& gate, int64_t act) {
   check_f32(y, "group_rmsnorm input");
   check_f32(w, "group_rmsnorm weight");
   TORCH_CHECK(y.dim() == 2 && groups >= 1 && y.size(1) % groups == 0 && w.numel() == y.size(1));
+  if (gate.has_value()) {
+    check_act(*gate, "group_rmsnorm gate");
+    TORCH_CHECK(gate->sizes() == y.sizes() && gate->stride(1) == 1, "group_rmsnorm: gate [rows, W] with a dense last axis");
+  }
   c10::cuda::CUDAGuard guard(y.device());
   auto out = at::empty(y.sizes(), y.options().dtype(out_lp ? at::kBFloat16 : at::kFloat));
   group_rmsnorm_launch(y.data_ptr<float>(), w.data_ptr<float>(), out.data_ptr(), out_lp, (int)y.size(0), (int)y.size(1), (int)groups, (float)eps,
+                       gate.has_value() ? gate->data_ptr() : nullptr, gate.has_value() ? gate->stride(0) : 0, gate.has_value() && is_lp(*gate), (int)act,
                        stream());
   return out;
 }
@@ -354,10 +532,10 @@ void head_gate_mul(at::Tensor x, const at::Tensor& gate) {
 
 at::Tensor gated_act_mul(const at::Tensor& gate, const at::Tensor& other, int64_t act, bool on_other) {
   check_act(gate, "gated_act_mul gate");
-  TORCH_CHECK(gate.dim() == 2 && gate.is_contiguous() && other.is_cuda() && other.scalar_type() == gate.scalar_type() && other.dim() == 2 &&
+  TORCH_CHECK(gate.dim() == 2 && gate.stride(1) == 1 && other.is_cuda() && other.scalar_type() == gate.scalar_type() && other.dim() == 2 &&
               other.sizes() == gate.sizes() && other.stride(1) == 1, "gated_act_mul: [rows, C] inputs of one type, the second with a row stride");
   c10::cuda::CUDAGuard guard(gate.device());
-  auto out = at::empty_like(gate);
+  auto out = at::empty(gate.sizes(), gate.options());
   gated_act_mul_launch(gate.data_ptr(), gate.stride(0), other.data_ptr(), other.stride(0), out.data_ptr(), gate.size(0), (int)gate.size(1), (int)act,
                        on_other, is_lp(gate), stream());
   return out;
@@ -375,7 +553,8 @@ at::Tensor unary_act(const at::Tensor& x, int64_t act) {
 // Routed two-matrix experts: x [N, H], w_up [E, I, H], w_down [E, H, I] (activation type), topk_w fp32 / topk_i int32 [N, k].
 // `tc`: bf16 with H and I in multiples of 64 -> grouped tcgen05 GEMMs, the activation as an elementwise pass between them.
 at::Tensor moe_plain(const at::Tensor& x, const at::Tensor& w_up, const at::Tensor& w_down, const at::Tensor& topk_w, const at::Tensor& topk_i,
-                     int64_t expert_offset, int64_t act, bool tc, bool gated) {
+                     int64_t expert_offset, int64_t act, bool tc, bool gated, double limit, double alpha) {
+  TORCH_CHECK(act != 7 || gated, "moe_plain: the clamped gate product needs gated experts");
   check_act(x, "moe_plain x");
   TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && w_up.dim() == 3 && w_down.dim() == 3 && w_up.is_contiguous() && w_down.is_contiguous() &&
               w_up.scalar_type() == x.scalar_type() && w_down.scalar_type() == x.scalar_type() && w_up.is_cuda() && w_down.is_cuda());
@@ -393,7 +572,7 @@ at::Tensor moe_plain(const at::Tensor& x, const at::Tensor& w_up, const at::Tens
   if (N * k <= 32) {        // decode steps: weight-streaming kernels, no permutation
     auto h = at::empty({(int64_t)N * k, I}, x.options());
     moe_plain_decode_launch(x.data_ptr(), w_up.data_ptr(), w_down.data_ptr(), topk_w.data_ptr<float>(), topk_i.data_ptr<int>(), h.data_ptr(),
-                            out.data_ptr(), N, k, H, I, (int)expert_offset, E, (int)act, gated, lp, st);
+                            out.data_ptr(), N, k, H, I, (int)expert_offset, E, (int)act, gated, (float)limit, (float)alpha, lp, st);
     return out;
   }
   const int64_t R = (((int64_t)N * k + (int64_t)E * 127) + 127) / 128 * 128;   // static bound: graph-stable shapes
@@ -418,7 +597,7 @@ at::Tensor moe_plain(const at::Tensor& x, const at::Tensor& w_up, const at::Tens
   if (gated) {
     auto gu = at::empty({R, 2 * (int64_t)I}, x.options());
     moe_plain_gemm_launch(xp.data_ptr(), w_up.data_ptr(), gu.data_ptr(), (int)R, 2 * I, H, 0, tile_expert.data_ptr<int>(), lp, st);
-    moe_plain_gate_mul_launch(gu.data_ptr(), h.data_ptr(), (int)R, I, (int)act, tile_expert.data_ptr<int>(), lp, st);
+    moe_plain_gate_mul_launch(gu.data_ptr(), h.data_ptr(), (int)R, I, (int)act, (float)limit, (float)alpha, tile_expert.data_ptr<int>(), lp, st);
   } else {
     moe_plain_gemm_launch(xp.data_ptr(), w_up.data_ptr(), h.data_ptr(), (int)R, I, H, (int)act, tile_expert.data_ptr<int>(), lp, st);
   }
@@ -566,18 +745,18 @@ std::tuple<at::Tensor, OptT> stream_sandwich_norm(const at::Tensor& x, const Opt
 
 at::Tensor head_norm_rope_append(const at::Tensor& pr, int64_t n_q, int64_t n_kv, int64_t D, int64_t Dv, const OptT& cos, const OptT& sin,
                                  const OptT& q_w, const OptT& k_w, int64_t norm_at, double eps, bool value_from_key, at::Tensor k_cache,
-                                 at::Tensor v_cache, const at::Tensor& block_table, const at::Tensor& ctx, const at::Tensor& qlen) {
+                                 at::Tensor v_cache, const at::Tensor& block_table, const at::Tensor& ctx, const at::Tensor& qlen, int64_t n_v) {
   check_act(pr, "head_norm_rope_append rows");
   check_rows(pr, "head_norm_rope_append rows");
   const int64_t B = pr.size(0), T = pr.size(1);
-  const int64_t need = n_q * D + n_kv * D + (value_from_key ? 0 : n_kv * Dv);
+  const int64_t need = n_q * D + n_kv * D + (value_from_key ? 0 : n_v * Dv);
   TORCH_CHECK(pr.size(2) >= need && D >= 1 && D <= 256 && Dv >= 1 && (!value_from_key || Dv == D), "head_norm_rope_append: q | k | v slices, head size <= 256");
-  TORCH_CHECK(norm_at >= 0 && norm_at <= 2);
+  TORCH_CHECK(norm_at >= 0 && norm_at <= 2 && n_v >= 1 && (!value_from_key || n_v == n_kv));
   TORCH_CHECK(k_cache.is_cuda() && k_cache.scalar_type() == pr.scalar_type() && k_cache.is_contiguous() && k_cache.dim() == 4 &&
               k_cache.size(2) == n_kv && k_cache.size(3) == D, "head_norm_rope_append: key cache [blocks, page, kv heads, D]");
   TORCH_CHECK(v_cache.is_cuda() && v_cache.scalar_type() == pr.scalar_type() && v_cache.is_contiguous() && v_cache.dim() == 4 &&
-              v_cache.size(0) == k_cache.size(0) && v_cache.size(1) == k_cache.size(1) && v_cache.size(2) == n_kv && v_cache.size(3) == Dv,
-              "head_norm_rope_append: value cache [blocks, page, kv heads, Dv]");
+              v_cache.size(0) == k_cache.size(0) && v_cache.size(1) == k_cache.size(1) && v_cache.size(2) == n_v && v_cache.size(3) == Dv,
+              "head_norm_rope_append: value cache [blocks, page, value heads, Dv]");
   TORCH_CHECK(block_table.is_cuda() && block_table.scalar_type() == at::kInt && block_table.is_contiguous() && block_table.dim() == 2 &&
               block_table.size(0) == B);
   check_i32(ctx, B, "ctx_len");
@@ -596,7 +775,7 @@ at::Tensor head_norm_rope_append(const at::Tensor& pr, int64_t n_q, int64_t n_kv
   p.p = pr.data_ptr(); p.p_sb = pr.stride(0); p.p_st = pr.stride(1);
   p.q_out = q.data_ptr(); p.k_cache = k_cache.data_ptr(); p.v_cache = v_cache.data_ptr();
   p.block_table = block_table.data_ptr<int>(); p.ctx_len = ctx.data_ptr<int>(); p.q_len = qlen.data_ptr<int>();
-  p.B = (int)B; p.T = (int)T; p.n_q = (int)n_q; p.n_kv = (int)n_kv; p.D = (int)D; p.Dv = (int)Dv; p.page = (int)k_cache.size(1);
+  p.B = (int)B; p.T = (int)T; p.n_q = (int)n_q; p.n_kv = (int)n_kv; p.n_v = (int)n_v; p.D = (int)D; p.Dv = (int)Dv; p.page = (int)k_cache.size(1);
   p.max_blocks = (int)block_table.size(1); p.norm_at = (int)norm_at; p.value_from_key = value_from_key ? 1 : 0; p.eps = (float)eps;
   head_norm_rope_append_launch(p, is_lp(pr), stream());
   return q;
@@ -654,6 +833,12 @@ void register_seqmix(pybind11::module_& m) {
   m.def("head_norm_rope_append", &head_norm_rope_append);
   m.def("gated_delta_scan", &gated_delta_scan);
   m.def("head_rmsnorm_gate", &head_rmsnorm_gate);
+  m.def("stream_mix_norm_conv", &stream_mix_norm_conv);
+  m.def("paged_diff_attention", &paged_diff_attention);
+  m.def("delta_front", &delta_front);
+  m.def("channel_delta_scan", &channel_delta_scan);
+  m.def("decay_scan", &decay_scan);
+  m.def("table_route", &table_route);
   m.def("router_topk", &router_topk);
   m.def("rope_half_tail", &rope_half_tail);
   m.def("stream_norm_conv", &stream_norm_conv);
