@@ -75,7 +75,8 @@ class BalivikInferenceConfig(InferenceConfig):
         for i, layer in enumerate(d["layers"]):
             if layer["type"] == "channel_delta":           # the ranks stand in the tensors' shapes only
                 for name, tensor in (("decay_rank", "a1"), ("gate_rank", "g1")):
-                    layer["mixer"].setdefault(name, shapes[f"l{i}.mix.{tensor}"][0])
+                    if f"l{i}.mix.{tensor}" in shapes:
+                        layer["mixer"][name] = shapes[f"l{i}.mix.{tensor}"][0]
 
         def load(self):
             for k, v in d.items():
