@@ -364,6 +364,240 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
     }
 }
 
+// ---- fixed decays, chunked form on tensor cores (bf16 rows, key sizes 64 / 128): prompt portions ------------------------------------------
+// Block = (batch row, head, 32 value channels), 4 warps; time runs in chunks of 64 steps.  With q, k, v after SiLU (bf16) and the state M (fp32,
+// in accumulator registers, [value, key]) before the chunk, for steps t, s counted inside the chunk of n live steps:
+//     y_t = decay^(t+1) M q_t + sum_{s <= t} decay^(t-s) (q_t . k_s) v_s
+//     M   = decay^n M + sum_s decay^(n-1-s) v_s k_s^T
+// All products run on mma.sync m16n8k16 with fp32 accumulators.  The operands that are fp32 by nature — the state, the decayed scores and the
+// decayed values — enter as a bf16 pair (value, remainder), two products each, so that they keep 16 bits.  Raw rows arrive through cp.async
+// one chunk ahead; a thread applies SiLU in place to the pieces it copied itself.
+constexpr int CS_C = 64, CS_NV = 32, CS_THREADS = 128, CS_MIN_T = 16;
+
+__device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16(a, b);
+  lo = pack_bf16(a - bf16lo(hi), b - bf16hi(hi));
+}
+__device__ __forceinline__ float silu_fast(float v) { return __fdividef(v, 1.f + __expf(-v)); }
+
+template <int D>
+__global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearScanParams p) {
+  extern __shared__ __align__(16) unsigned char csm[];
+  constexpr int DS = D + 8, VS = CS_NV + 8, STAGE = 2 * CS_C * DS + CS_C * VS, NTW = D / 32;
+  __nv_bfloat16* stage0 = reinterpret_cast<__nv_bfloat16*>(csm);           // two stages of q [64][DS], k [64][DS], v [64][VS]
+  __nv_bfloat16* Sh = stage0 + 2 * STAGE;                                  // state [32][DS]: value, then remainder
+  __nv_bfloat16* Sl = Sh + CS_NV * DS;
+  __nv_bfloat16* Wh = Sl + CS_NV * DS;                                     // decayed values [64][VS]: value, then remainder
+  __nv_bfloat16* Wl = Wh + CS_C * VS;
+  float* pw = reinterpret_cast<float*>(Wl + CS_C * VS);                    // powers of the decay, 0 .. 64
+  const int b = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * CS_NV, Dv = p.Dv;
+  const int n_tok = p.q_len[b];
+  if (n_tok <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tig = lane & 3;
+  const __nv_bfloat16* xrow = (const __nv_bfloat16*)p.x + (long long)b * p.x_sb;
+  const int Cq = p.nh * D;
+  float* Sg = p.state + ((long long)p.lines[b] * p.nh + h) * Dv * D;
+  if (tid <= CS_C) pw[tid] = powf(p.decay[h], (float)tid);
+  // this warp's share of the state: all 32 value channels x key channels [warp * D / 4, + D / 4)
+  float S[2][NTW][4];
+  const bool has_ctx = p.ctx_len[b] > 0;
+#pragma unroll
+  for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < NTW; ++nt)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int v = p0 + mt * 16 + gid + r * 8, d = warp * (D / 4) + nt * 8 + tig * 2;
+        float2 s = make_float2(0.f, 0.f);
+        if (has_ctx && v < Dv) s = *reinterpret_cast<const float2*>(Sg + (long long)v * D + d);
+        S[mt][nt][r * 2] = s.x;
+        S[mt][nt][r * 2 + 1] = s.y;
+      }
+  constexpr int QP = CS_C * D / 8 / CS_THREADS, VP = CS_C * CS_NV / 8 / CS_THREADS;        // 16-byte pieces per thread
+  auto issue = [&](int t0, int st) {
+    __nv_bfloat16* qd = stage0 + st * STAGE;
+    __nv_bfloat16* kd = qd + CS_C * DS;
+    __nv_bfloat16* vd = kd + CS_C * DS;
+    const int n = min(CS_C, n_tok - t0);
+#pragma unroll
+    for (int i = 0; i < QP; ++i) {
+      const int c = tid + i * CS_THREADS, t = c / (D / 8), d = (c % (D / 8)) * 8;
+      const bool on = t < n;
+      const __nv_bfloat16* q = on ? xrow + (long long)(t0 + t) * p.x_st + h * D + d : xrow;
+      cp_async16(qd + t * DS + d, q, on);
+      cp_async16(kd + t * DS + d, on ? q + Cq : q, on);
+    }
+#pragma unroll
+    for (int i = 0; i < VP; ++i) {
+      const int c = tid + i * CS_THREADS, t = c / (CS_NV / 8), v = (c % (CS_NV / 8)) * 8;
+      const bool on = t < n && p0 + v < Dv;
+      cp_async16(vd + t * VS + v, on ? xrow + (long long)(t0 + t) * p.x_st + 2 * Cq + h * Dv + p0 + v : xrow, on);
+    }
+    cp_async_commit();
+  };
+  auto silu_piece = [&](__nv_bfloat16* at, float* f) {
+    uint4 r = *reinterpret_cast<const uint4*>(at);
+    f[0] = bf16lo(r.x); f[1] = bf16hi(r.x); f[2] = bf16lo(r.y); f[3] = bf16hi(r.y);
+    f[4] = bf16lo(r.z); f[5] = bf16hi(r.z); f[6] = bf16lo(r.w); f[7] = bf16hi(r.w);
+    if (p.silu) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] = silu_fast(f[e]);
+      r = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+      *reinterpret_cast<uint4*>(at) = r;
+      f[0] = bf16lo(r.x); f[1] = bf16hi(r.x); f[2] = bf16lo(r.y); f[3] = bf16hi(r.y);
+      f[4] = bf16lo(r.z); f[5] = bf16hi(r.z); f[6] = bf16lo(r.w); f[7] = bf16hi(r.w);
+    }
+  };
+  issue(0, 0);
+  __syncthreads();                              // pw is there
+  int st = 0;
+  for (int t0 = 0; t0 < n_tok; t0 += CS_C, st ^= 1) {
+    const int n = min(CS_C, n_tok - t0);
+    __nv_bfloat16* Q = stage0 + st * STAGE;
+    __nv_bfloat16* K = Q + CS_C * DS;
+    __nv_bfloat16* V = K + CS_C * DS;
+    cp_async_wait<0>();
+    {
+      float f[8];
+#pragma unroll 2
+      for (int i = 0; i < QP; ++i) {
+        const int c = tid + i * CS_THREADS, t = c / (D / 8), d = (c % (D / 8)) * 8;
+        silu_piece(Q + t * DS + d, f);
+        silu_piece(K + t * DS + d, f);
+      }
+#pragma unroll
+      for (int i = 0; i < VP; ++i) {
+        const int c = tid + i * CS_THREADS, t = c / (CS_NV / 8), v = (c % (CS_NV / 8)) * 8;
+        silu_piece(V + t * VS + v, f);
+        const float w = t < n ? pw[n - 1 - t] : 0.f;
+        uint4 hi, lo;
+        split_bf16(f[0] * w, f[1] * w, hi.x, lo.x); split_bf16(f[2] * w, f[3] * w, hi.y, lo.y);
+        split_bf16(f[4] * w, f[5] * w, hi.z, lo.z); split_bf16(f[6] * w, f[7] * w, hi.w, lo.w);
+        *reinterpret_cast<uint4*>(Wh + t * VS + v) = hi;
+        *reinterpret_cast<uint4*>(Wl + t * VS + v) = lo;
+      }
+    }
+#pragma unroll
+    for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+      for (int nt = 0; nt < NTW; ++nt)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int at = (mt * 16 + gid + r * 8) * DS + warp * (D / 4) + nt * 8 + tig * 2;
+          uint32_t hi, lo;
+          split_bf16(S[mt][nt][r * 2], S[mt][nt][r * 2 + 1], hi, lo);
+          *reinterpret_cast<uint32_t*>(Sh + at) = hi;
+          *reinterpret_cast<uint32_t*>(Sl + at) = lo;
+        }
+    __syncthreads();
+    if (t0 + CS_C < n_tok) issue(t0 + CS_C, st ^ 1);          // the other stage was last read before this barrier
+    const int r0 = warp * 16 + gid, r1 = r0 + 8;              // this thread's two steps
+    if (warp * 16 < n) {
+      float o[CS_NV / 8][4], sc[CS_C / 8][4];
+#pragma unroll
+      for (int i = 0; i < CS_NV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+#pragma unroll
+      for (int i = 0; i < CS_C / 8; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < D / 16; ++ks) {
+        const __nv_bfloat16* qp = Q + r0 * DS + ks * 16 + tig * 2;
+        const uint32_t qa[4] = {*reinterpret_cast<const uint32_t*>(qp), *reinterpret_cast<const uint32_t*>(qp + 8 * DS),
+                                *reinterpret_cast<const uint32_t*>(qp + 8), *reinterpret_cast<const uint32_t*>(qp + 8 * DS + 8)};
+#pragma unroll
+        for (int nt = 0; nt < CS_NV / 8; ++nt) {
+          const int at = (nt * 8 + gid) * DS + ks * 16 + tig * 2;
+          const uint32_t bh[2] = {*reinterpret_cast<const uint32_t*>(Sh + at), *reinterpret_cast<const uint32_t*>(Sh + at + 8)};
+          const uint32_t bl[2] = {*reinterpret_cast<const uint32_t*>(Sl + at), *reinterpret_cast<const uint32_t*>(Sl + at + 8)};
+          mma_bf16_16816(o[nt], qa, bh);
+          mma_bf16_16816(o[nt], qa, bl);
+        }
+#pragma unroll
+        for (int nt = 0; nt < CS_C / 8; ++nt)
+          if (nt <= 2 * warp + 1) {                           // later steps than this warp's last one are not seen
+            const __nv_bfloat16* kp = K + (nt * 8 + gid) * DS + ks * 16 + tig * 2;
+            const uint32_t bb[2] = {*reinterpret_cast<const uint32_t*>(kp), *reinterpret_cast<const uint32_t*>(kp + 8)};
+            mma_bf16_16816(sc[nt], qa, bb);
+          }
+      }
+      const float d0 = pw[r0 + 1], d1 = pw[r1 + 1];
+#pragma unroll
+      for (int i = 0; i < CS_NV / 8; ++i) { o[i][0] *= d0; o[i][1] *= d0; o[i][2] *= d1; o[i][3] *= d1; }
+#pragma unroll
+      for (int kk = 0; kk < CS_C / 16; ++kk)
+        if (kk <= warp) {
+          uint32_t ah[4], al[4];
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int nt = kk * 2 + half, s = nt * 8 + tig * 2;
+            float f[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int gap = (e < 2 ? r0 : r1) - (s + (e & 1));
+              f[e] = gap >= 0 ? sc[nt][e] * pw[gap] : 0.f;
+            }
+            split_bf16(f[0], f[1], ah[half * 2], al[half * 2]);
+            split_bf16(f[2], f[3], ah[half * 2 + 1], al[half * 2 + 1]);
+          }
+#pragma unroll
+          for (int nv = 0; nv < CS_NV / 8; nv += 2) {
+            uint32_t r[4];
+            ldmatrix_x4_trans(r, V + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VS + (nv + (lane >> 4)) * 8);
+            const uint32_t ba[2] = {r[0], r[1]}, bb[2] = {r[2], r[3]};
+            mma_bf16_16816(o[nv], ah, ba);
+            mma_bf16_16816(o[nv], al, ba);
+            mma_bf16_16816(o[nv + 1], ah, bb);
+            mma_bf16_16816(o[nv + 1], al, bb);
+          }
+        }
+      float* y = p.y + ((long long)b * p.T + t0) * p.nh * Dv + h * Dv + p0;
+#pragma unroll
+      for (int nv = 0; nv < CS_NV / 8; ++nv) {
+        const int col = nv * 8 + tig * 2;
+        if (p0 + col < Dv) {
+          if (r0 < n) *reinterpret_cast<float2*>(y + (long long)r0 * p.nh * Dv + col) = make_float2(o[nv][0], o[nv][1]);
+          if (r1 < n) *reinterpret_cast<float2*>(y + (long long)r1 * p.nh * Dv + col) = make_float2(o[nv][2], o[nv][3]);
+        }
+      }
+    }
+    // state after the chunk
+    const float dn = pw[n];
+#pragma unroll
+    for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+      for (int nt = 0; nt < NTW; ++nt) { S[mt][nt][0] *= dn; S[mt][nt][1] *= dn; S[mt][nt][2] *= dn; S[mt][nt][3] *= dn; }
+#pragma unroll
+    for (int kk = 0; kk < CS_C / 16; ++kk) {
+      uint32_t kb[NTW / 2][4];
+#pragma unroll
+      for (int nt = 0; nt < NTW; nt += 2)
+        ldmatrix_x4_trans(kb[nt / 2], K + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * DS + warp * (D / 4) + (nt + (lane >> 4)) * 8);
+#pragma unroll
+      for (int mt = 0; mt < 2; ++mt) {
+        uint32_t wh[4], wl[4];
+        const int at = (kk * 16 + (lane & 7) + (lane >> 4) * 8) * VS + mt * 16 + ((lane >> 3) & 1) * 8;
+        ldmatrix_x4_trans(wh, Wh + at);
+        ldmatrix_x4_trans(wl, Wl + at);
+#pragma unroll
+        for (int nt = 0; nt < NTW; ++nt) {
+          const uint32_t bb[2] = {kb[nt / 2][(nt & 1) * 2], kb[nt / 2][(nt & 1) * 2 + 1]};
+          mma_bf16_16816(S[mt][nt], wh, bb);
+          mma_bf16_16816(S[mt][nt], wl, bb);
+        }
+      }
+    }
+    __syncthreads();                            // the state and decayed-value copies are rewritten at the top of the next chunk
+  }
+#pragma unroll
+  for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < NTW; ++nt)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int v = p0 + mt * 16 + gid + r * 8, d = warp * (D / 4) + nt * 8 + tig * 2;
+        if (v < Dv) *reinterpret_cast<float2*>(Sg + (long long)v * D + d) = make_float2(S[mt][nt][r * 2], S[mt][nt][r * 2 + 1]);
+      }
+}
+
 __global__ void __launch_bounds__(256) table_route_kernel(const int* __restrict__ table, const int* __restrict__ ids, const int* __restrict__ q_len,
                                                           float* __restrict__ w, int* __restrict__ idx, int B, int T, int k, int vocab) {
   const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
@@ -442,6 +676,20 @@ void channel_delta_scan_launch(const LinearScanParams& p, cudaStream_t st) {
 void decay_scan_launch(const LinearScanParams& p, bool lp, cudaStream_t st) {
   if (p.B <= 0 || p.T <= 0) return;
   if (p.D > 256 || p.n_qk != p.nh) throw std::runtime_error("decay_scan: key size <= 256");
+  if (lp && p.T >= CS_MIN_T && (p.D == 64 || p.D == 128) && p.Dv % 8 == 0 && p.x_st % 8 == 0 && p.x_sb % 8 == 0 &&
+      (((uintptr_t)p.x | (uintptr_t)p.state | (uintptr_t)p.y) & 15) == 0) {
+    // prompt portions in bf16: chunks on tensor cores
+    const dim3 grid((p.Dv + CS_NV - 1) / CS_NV, p.nh, p.B);
+    auto go = [&](auto d) {
+      constexpr int D = decltype(d)::value;
+      const size_t smem = sizeof(__nv_bfloat16) * (2 * (2 * CS_C * (D + 8) + CS_C * (CS_NV + 8)) + 2 * CS_NV * (D + 8) + 2 * CS_C * (CS_NV + 8)) +
+                          sizeof(float) * (CS_C + 1);
+      opt_in(decay_scan_chunk_kernel<D>, smem);
+      decay_scan_chunk_kernel<D><<<grid, CS_THREADS, smem, st>>>(p);
+    };
+    if (p.D == 64) go(std::integral_constant<int, 64>{}); else go(std::integral_constant<int, 128>{});
+    return;
+  }
   const bool aligned = p.D % 4 == 0 && ((uintptr_t)p.state & 15) == 0;
   if (lp) scan_go<__nv_bfloat16, false>(p, aligned, st); else scan_go<float, false>(p, aligned, st);
 }
