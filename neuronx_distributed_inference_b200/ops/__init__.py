@@ -738,7 +738,7 @@ def stream_mix_norm_conv(x, y, mix, out_w, in_w, norm_w, conv_w, state, slots, c
     S, W = in_w.shape[0], x.shape[-1]
     taps = 1 if conv_w is None else conv_w.shape[1]
     if (_use_cuda(x) and x.dtype == torch.float32 and (y is None or y.dtype in _MIX_DTYPES) and S <= _MIX_MAX_STREAMS and taps <= _MIX_MAX_TAPS
-            and W <= 16384 and (state is None or state.dtype == torch.float32)):
+            and taps * W <= 51200 and (state is None or state.dtype == torch.float32)):
         stats["stream_mix_norm_conv"] += 1
         f32 = lambda t: None if t is None else t.float().contiguous()          # noqa: E731
         i32 = lambda t: None if t is None else _i32(t)                         # noqa: E731
