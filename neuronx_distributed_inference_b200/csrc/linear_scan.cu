@@ -255,7 +255,7 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
   for (int t0 = 0; t0 < n_tok; t0 += LS_TT, st ^= 1) {
     const int tt = min(LS_TT, n_tok - t0);
     if constexpr (DELTA && ALIGNED) cp_async_wait<0>();
-    __syncthreads();                            // this round has landed; everyone is done with the other stage, kq, bt and os
+    __syncthreads();                            // these steps have landed; everyone is done with the other stage, kq, bt and os
     const float* qs = lsm + st * STAGE;
     const float* ks = qs + LS_TT * DP;
     const float* gs = ks + LS_TT * DP;

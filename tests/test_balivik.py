@@ -689,7 +689,7 @@ def test_gpu_prompt_portions_over_a_prefix_match_the_plain_maps():
     from neuronx_distributed_inference_b200 import ops
     g = torch.Generator().manual_seed(9)
     H, G, page, lam, diff = 4, 2, 16, 0.6, 0.3
-    for D, Dv in ((64, 64), (64, 128), (128, 128), (48, 96)):
+    for D, Dv in ((64, 64), (64, 128), (128, 128), (40, 72)):
         ctx, ql, T, nblk = (37, 0, 130), (100, 61, 1), 100, 16
         k, v = torch.randn(3, 240, G, 2, D, generator=g), torch.randn(3, 240, G, Dv, generator=g)
         q = torch.randn(3, T, H, 2, D, generator=g)
