@@ -2,6 +2,7 @@
 //   * the gated delta rule with one decay per head and key channel, and the kernel that makes its rows (convolution, SiLU, unit norms,
 //     decays, write strengths);
 //   * linear attention with a fixed decay per head;
+//   * matrix memory with exponential input gates, a running maximum and a key sum as denominator;
 // and routing by token id.  States, decays, unit norms and everything else inside a recurrence are fp32; compiled WITHOUT fast-math.
 #include <cuda_bf16.h>
 #include <math.h>
@@ -174,19 +175,34 @@ __global__ void __launch_bounds__(FRONT_WARPS * 32) delta_front_kernel(DeltaFron
 //   delta: s <- decay * s per key channel; r = s . k, o = s . q on the shrunk state share one lane reduction; u = beta (v - r); s += u k;
 //          o += u (k . q), k . q formed once per step and round
 //   fixed: s <- decay_h s + v k;  o = s . q
+//   gated: s <- fade_t s + (put_t v) k;  o = s . q / den_t.  A third warp of the block forms the gates one round ahead (running maximum step by
+//          step), keeps the key sum n and the denominators den_t = max(|n . q|, exp(-m)) + 1e-6
+constexpr int LS_FIXED = 0, LS_DELTA = 1, LS_GATED = 2;
+constexpr float MLSTM_DEN_EPS = 1e-6f;
 constexpr int LS_PT = 16, LS_TT = 16, LS_NS = 8, LS_CPT = 2, LS_THREADS = (LS_PT / LS_CPT) * LS_NS;
 
-template <typename T, bool DELTA, int NJ, bool ALIGNED>
-__global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParams p) {
+// capped log input gate and log forget gate
+__device__ __forceinline__ float2 log_gates(float i, float f, float cap) {
+  const float z = cap * tanhf(f / cap);
+  return make_float2(cap * tanhf(i / cap), fminf(z, 0.f) - log1pf(expf(-fabsf(z))));
+}
+
+template <typename T, int KIND, int NJ, bool ALIGNED>
+__global__ void __launch_bounds__(LS_THREADS + (KIND == LS_GATED ? 32 : 0)) linear_scan_kernel(LinearScanParams p) {
   extern __shared__ __align__(16) float lsm[];
+  constexpr bool DELTA = KIND == LS_DELTA, GATED = KIND == LS_GATED;
+  constexpr int NT = LS_THREADS + (GATED ? 32 : 0);
   constexpr int DP = NJ * 32, ROWS = DELTA ? 3 : 2, STAGE = ROWS * LS_TT * DP + LS_TT * LS_PT;
   float* kq = lsm + 2 * STAGE;                  // [TT] k . q
   float* bt = kq + LS_TT;                       // [TT] beta
   float* os = bt + LS_TT;                       // [TT][PT]
+  float* gts = os + LS_TT * LS_PT;              // gated: two stages of fade, put, exp(-m) [TT] each, then the denominators [TT]
+  float* den = gts + 6 * LS_TT;
   const int D = p.D, Dv = p.Dv, b = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * LS_PT;
   const int n_tok = p.q_len[b];
   if (n_tok <= 0) return;
   const int tid = threadIdx.x, pl = tid / LS_NS, ns = tid % LS_NS;
+  const bool channels = !GATED || tid < LS_THREADS;      // false: the warp of gates and key sum
   const int gq = h / (p.nh / p.n_qk), Cq = p.n_qk * D;
   float* Sg = p.state + ((long long)p.lines[b] * p.nh + h) * Dv * D;
   const bool has_ctx = p.ctx_len[b] > 0;
@@ -197,7 +213,7 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
     for (int j = 0; j < NJ; ++j) {
       const int d = j * 32 + ns * 4, pc = p0 + pl * LS_CPT + c;
       S[c][j] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (has_ctx && pc < Dv) {
+      if (has_ctx && channels && pc < Dv) {
         const float* s = Sg + (long long)pc * D + d;
         if (ALIGNED) { if (d < D) S[c][j] = *reinterpret_cast<const float4*>(s); }
         else {
@@ -209,7 +225,46 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
       }
     }
   const T* xrow = (const T*)p.x + (long long)b * p.x_sb;
-  const float lam = DELTA ? 0.f : p.decay[h];
+  const float lam = KIND == LS_FIXED ? p.decay[h] : 0.f;
+  // gated: this block's copy of the key sum (lane + 32 j of the third warp) and of the running maximum
+  float nk[GATED ? NJ : 1], m_run = 0.f, i_b = 0.f, f_b = 0.f;
+  const float q_scale = rsqrtf((float)D);
+  const long long copy = (((long long)p.lines[b] * p.nh + h) * gridDim.x + blockIdx.x);
+  auto gates = [&](int t0, int st) {
+    const int lane = tid & 31, tt = min(LS_TT, n_tok - t0);
+    float2 g = make_float2(0.f, 0.f);
+    if (lane < tt) {
+      const T* r = (const T*)p.x + (long long)b * p.x_sb + (long long)(t0 + lane) * p.x_st + p.gate_at + h;
+      g = log_gates(ldf1(r) + i_b, ldf1(r + p.nh) + f_b, p.cap);
+    }
+    float before = 0.f, after = 0.f;
+#pragma unroll 1
+    for (int t = 0; t < tt; ++t) {
+      const float it = __shfl_sync(0xffffffffu, g.x, t), ft = __shfl_sync(0xffffffffu, g.y, t);
+      const float m = fmaxf(ft + m_run, it);
+      if (lane == t) { before = m_run; after = m; }
+      m_run = m;
+    }
+    if (lane < tt) {
+      float* d = gts + st * 3 * LS_TT + lane;
+      d[0] = expf(g.y + before - after);
+      d[LS_TT] = expf(g.x - after);
+      d[2 * LS_TT] = expf(-after);
+    }
+  };
+  if constexpr (GATED) {
+    if (!channels) {
+      i_b = p.i_bias[h];
+      f_b = p.f_bias[h];
+      if (has_ctx) m_run = p.run_max[copy];
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const int d = (tid & 31) + 32 * j;
+        nk[j] = has_ctx && d < D ? p.key_sum[copy * D + d] : 0.f;
+      }
+      gates(0, 0);
+    }
+  }
   // rows of steps t0 .. into stage st; zeros past the key channels and past the live steps
   auto issue = [&](int t0, int st) {
     const int tt = min(LS_TT, n_tok - t0);
@@ -219,7 +274,7 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
     float* vd = qd + ROWS * LS_TT * DP;
     if constexpr (DELTA && ALIGNED) {
       constexpr int CPR = DP / 4;
-      for (int i = tid; i < LS_TT * CPR; i += LS_THREADS) {
+      for (int i = tid; i < LS_TT * CPR; i += NT) {
         const int t = i / CPR, d = (i % CPR) * 4, at = t * DP + d;
         const bool on = t < tt && d < D;
         const float* q = on ? (const float*)xrow + (long long)(t0 + t) * p.x_st + gq * D + d : (const float*)xrow;
@@ -227,16 +282,16 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
         cp_async16(kd + at, on ? q + Cq : q, on);
         cp_async16(gd + at, on ? p.decay + ((long long)b * p.T + t0 + t) * p.nh * D + h * D + d : (const float*)xrow, on);
       }
-      for (int i = tid; i < LS_TT * (LS_PT / 4); i += LS_THREADS) {
+      for (int i = tid; i < LS_TT * (LS_PT / 4); i += NT) {
         const int t = i / (LS_PT / 4), c = (i % (LS_PT / 4)) * 4;
         const bool on = t < tt && p0 + c < Dv;
         cp_async16(vd + t * LS_PT + c, on ? (const float*)xrow + (long long)(t0 + t) * p.x_st + 2 * Cq + h * Dv + p0 + c : (const float*)xrow, on);
       }
       cp_async_commit();
     } else {
-      auto act = [&](float v) { return (!DELTA && p.silu) ? silu_acc(v) : v; };
+      auto act = [&](float v) { return (KIND == LS_FIXED && p.silu) ? silu_acc(v) : v; };
       const int tl = (t0 == 0 && tt < LS_TT) ? tt : LS_TT;          // a lone short round touches its live steps only
-      for (int i = tid; i < tl * DP; i += LS_THREADS) {
+      for (int i = tid; i < tl * DP; i += NT) {
         const int t = i / DP, d = i % DP;
         const bool on = t < tt && d < D;
         const T* r = xrow + (long long)(t0 + t) * p.x_st + gq * D + d;
@@ -244,7 +299,7 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
         kd[i] = on ? act(ldf1(r + Cq)) : 0.f;
         if (DELTA) gd[i] = on ? p.decay[((long long)b * p.T + t0 + t) * p.nh * D + h * D + d] : 0.f;
       }
-      for (int i = tid; i < tl * LS_PT; i += LS_THREADS) {
+      for (int i = tid; i < tl * LS_PT; i += NT) {
         const int t = i / LS_PT, c = p0 + i % LS_PT;
         vd[i] = (t < tt && c < Dv) ? act(ldf1(xrow + (long long)(t0 + t) * p.x_st + 2 * Cq + h * Dv + c)) : 0.f;
       }
@@ -281,8 +336,27 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
       __syncthreads();
     }
     if (t0 + LS_TT < n_tok) issue(t0 + LS_TT, st ^ 1);
+    const float* gt = gts + st * 3 * LS_TT;
+    if constexpr (GATED) {
+      if (!channels) {
 #pragma unroll 1
-    for (int t = 0; t < tt; ++t) {
+        for (int t = 0; t < tt; ++t) {
+          const float fade = gt[t], put = gt[LS_TT + t];
+          float dot = 0.f;
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) {
+            const int d = t * DP + (tid & 31) + 32 * j;
+            nk[j] = fade * nk[j] + put * ks[d];
+            dot += nk[j] * qs[d];
+          }
+          dot = warp_sum(dot);
+          if ((tid & 31) == 0) den[t] = fmaxf(fabsf(dot * q_scale), gt[2 * LS_TT + t]) + MLSTM_DEN_EPS;
+        }
+        if (t0 + LS_TT < n_tok) gates(t0 + LS_TT, st ^ 1);
+      }
+    }
+#pragma unroll 1
+    for (int t = 0; channels && t < tt; ++t) {
       const float4* Kt = reinterpret_cast<const float4*>(ks + t * DP) + ns;
       const float4* Qt = reinterpret_cast<const float4*>(qs + t * DP) + ns;
       float4 kv[NJ];
@@ -321,13 +395,19 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
           sq[c] += u * kqt;
         }
       } else {
+        float lt = lam;
+        if constexpr (GATED) {
+          lt = gt[t];
+#pragma unroll
+          for (int c = 0; c < LS_CPT; ++c) vt[c] *= gt[LS_TT + t];
+        }
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
           const float4 k4 = Kt[j * 8], qv = Qt[j * 8];
 #pragma unroll
           for (int c = 0; c < LS_CPT; ++c) {
-            S[c][j].x = lam * S[c][j].x + vt[c] * k4.x; S[c][j].y = lam * S[c][j].y + vt[c] * k4.y;
-            S[c][j].z = lam * S[c][j].z + vt[c] * k4.z; S[c][j].w = lam * S[c][j].w + vt[c] * k4.w;
+            S[c][j].x = lt * S[c][j].x + vt[c] * k4.x; S[c][j].y = lt * S[c][j].y + vt[c] * k4.y;
+            S[c][j].z = lt * S[c][j].z + vt[c] * k4.z; S[c][j].w = lt * S[c][j].w + vt[c] * k4.w;
             sq[c] += (S[c][j].x * qv.x + S[c][j].z * qv.z) + (S[c][j].y * qv.y + S[c][j].w * qv.w);
           }
         }
@@ -341,9 +421,20 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
         for (int c = 0; c < LS_CPT; ++c) os[t * LS_PT + pl * LS_CPT + c] = sq[c];
     }
     __syncthreads();
-    for (int i = tid; i < tt * LS_PT; i += LS_THREADS) {
+    for (int i = tid; i < tt * LS_PT; i += NT) {
       const int t = i / LS_PT, c = p0 + i % LS_PT;
-      if (c < Dv) p.y[((long long)b * p.T + t0 + t) * p.nh * Dv + h * Dv + c] = os[i];
+      if (c < Dv) p.y[((long long)b * p.T + t0 + t) * p.nh * Dv + h * Dv + c] = GATED ? os[i] * q_scale / den[t] : os[i];
+    }
+  }
+  if constexpr (GATED) {
+    if (!channels) {
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const int d = (tid & 31) + 32 * j;
+        if (d < D) p.key_sum[copy * D + d] = nk[j];
+      }
+      if ((tid & 31) == 0) p.run_max[copy] = m_run;
+      return;
     }
   }
 #pragma unroll
@@ -364,7 +455,7 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
     }
 }
 
-// ---- fixed decays, chunked form on tensor cores (bf16 rows, key sizes 64 / 128): prompt portions ------------------------------------------
+// ---- fixed decays and exponential gates, chunked form on tensor cores (bf16 rows, key sizes 64 / 128 / 256): prompt portions ---------------
 // Block = (batch row, head, 32 value channels), 4 warps; time runs in chunks of 64 steps.  With q, k, v after SiLU (bf16) and the state M (fp32,
 // in accumulator registers, [value, key]) before the chunk, for steps t, s counted inside the chunk of n live steps:
 //     y_t = decay^(t+1) M q_t + sum_{s <= t} decay^(t-s) (q_t . k_s) v_s
@@ -372,6 +463,11 @@ __global__ void __launch_bounds__(LS_THREADS) linear_scan_kernel(LinearScanParam
 // All products run on mma.sync m16n8k16 with fp32 accumulators.  The operands that are fp32 by nature — the state, the decayed scores and the
 // decayed values — enter as a bf16 pair (value, remainder), two products each, so that they keep 16 bits.  Raw rows arrive through cp.async
 // one chunk ahead; a thread applies SiLU in place to the pieces it copied itself.
+// GATED: the powers of the decay become weights from the gates.  With F_t the sum of the log forget gates of the chunk up to t, g_s = i_s - F_s
+// and x_t = max(m, max_{s <= t} g_s) (m: the running maximum before the chunk), the running maximum at t is F_t + x_t and
+//     decay^(t+1) -> exp(m - x_t);   decay^(t-s) -> exp(g_s - x_t);   decay^(n-1-s) -> exp(g_s - x_n);   decay^n -> exp(m - x_n)
+// (no exponent is positive).  The key sum n follows the state with the same weights, n_t . q_t = exp(m - x_t) n . q_t + the row sum of the
+// weighted scores, and y_t is divided by max(|n_t . q_t|, exp(-F_t - x_t)) + 1e-6.  Warp 0 forms the gates one chunk ahead.
 constexpr int CS_C = 64, CS_NV = 32, CS_THREADS = 128, CS_MIN_T = 16;
 
 __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
@@ -380,8 +476,8 @@ __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint3
 }
 __device__ __forceinline__ float silu_fast(float v) { return __fdividef(v, 1.f + __expf(-v)); }
 
-template <int D>
-__global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearScanParams p) {
+template <int D, bool GATED>
+__global__ void __launch_bounds__(CS_THREADS, D > 128 ? 1 : 2) linear_chunk_kernel(LinearScanParams p) {
   extern __shared__ __align__(16) unsigned char csm[];
   constexpr int DS = D + 8, VS = CS_NV + 8, STAGE = 2 * CS_C * DS + CS_C * VS, NTW = D / 32;
   __nv_bfloat16* stage0 = reinterpret_cast<__nv_bfloat16*>(csm);           // two stages of q [64][DS], k [64][DS], v [64][VS]
@@ -389,7 +485,9 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
   __nv_bfloat16* Sl = Sh + CS_NV * DS;
   __nv_bfloat16* Wh = Sl + CS_NV * DS;                                     // decayed values [64][VS]: value, then remainder
   __nv_bfloat16* Wl = Wh + CS_C * VS;
-  float* pw = reinterpret_cast<float*>(Wl + CS_C * VS);                    // powers of the decay, 0 .. 64
+  float* pw = reinterpret_cast<float*>(Wl + CS_C * VS);                    // fixed: powers of the decay, 0 .. 64
+  // gated: two stages of g, x, exp(m - x), exp(-F - x) [64] each, of exp(m - x_n) and x_n, and of the key sum [D]; then exp(g - x_n) [64]
+  float *gts = pw, *tot = gts + 8 * CS_C, *nsum = tot + 4, *wgt = nsum + 2 * D;
   const int b = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * CS_NV, Dv = p.Dv;
   const int n_tok = p.q_len[b];
   if (n_tok <= 0) return;
@@ -397,10 +495,63 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
   const __nv_bfloat16* xrow = (const __nv_bfloat16*)p.x + (long long)b * p.x_sb;
   const int Cq = p.nh * D;
   float* Sg = p.state + ((long long)p.lines[b] * p.nh + h) * Dv * D;
-  if (tid <= CS_C) pw[tid] = powf(p.decay[h], (float)tid);
+  const float q_scale = rsqrtf((float)D);
+  float m_run = 0.f, i_b = 0.f, f_b = 0.f;
+  const int slices = (Dv + MLSTM_SLICE - 1) / MLSTM_SLICE, sl0 = p0 / MLSTM_SLICE;
+  const long long copy = ((long long)p.lines[b] * p.nh + h) * slices + sl0;      // of this block; the next one is its too when it exists
+  auto gates = [&](int t0, int st) {
+    const int n = min(CS_C, n_tok - t0);
+    float *g = gts + st * 4 * CS_C, f_sum = 0.f, x_max = m_run;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int t = half * 32 + lane;
+      float2 lg = make_float2(0.f, 0.f);
+      if (t < n) {
+        const __nv_bfloat16* r = xrow + (long long)(t0 + t) * p.x_st + p.gate_at + h;
+        lg = log_gates(__bfloat162float(r[0]) + i_b, __bfloat162float(r[p.nh]) + f_b, p.cap);
+      }
+      float F = lg.y;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float v = __shfl_up_sync(0xffffffffu, F, o);
+        if (lane >= o) F += v;
+      }
+      F += f_sum;
+      const float gs = t < n ? lg.x - F : -INFINITY;
+      float x = gs;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float v = __shfl_up_sync(0xffffffffu, x, o);
+        if (lane >= o) x = fmaxf(x, v);
+      }
+      x = fmaxf(x, x_max);
+      g[t] = gs;
+      g[CS_C + t] = x;
+      g[2 * CS_C + t] = expf(m_run - x);
+      g[3 * CS_C + t] = expf(-(F + x));
+      f_sum = __shfl_sync(0xffffffffu, F, 31);
+      x_max = __shfl_sync(0xffffffffu, x, 31);
+    }
+    if (lane == 0) {
+      tot[st * 2] = expf(m_run - x_max);
+      tot[st * 2 + 1] = x_max;
+    }
+    m_run = f_sum + x_max;
+  };
   // this warp's share of the state: all 32 value channels x key channels [warp * D / 4, + D / 4)
   float S[2][NTW][4];
   const bool has_ctx = p.ctx_len[b] > 0;
+  if constexpr (GATED) {
+    for (int d = tid; d < D; d += CS_THREADS) nsum[d] = has_ctx ? p.key_sum[copy * D + d] : 0.f;
+    if (warp == 0) {
+      i_b = p.i_bias[h];
+      f_b = p.f_bias[h];
+      if (has_ctx) m_run = p.run_max[copy];
+      gates(0, 0);
+    }
+  } else {
+    if (tid <= CS_C) pw[tid] = powf(p.decay[h], (float)tid);
+  }
 #pragma unroll
   for (int mt = 0; mt < 2; ++mt)
 #pragma unroll
@@ -439,7 +590,7 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
     uint4 r = *reinterpret_cast<const uint4*>(at);
     f[0] = bf16lo(r.x); f[1] = bf16hi(r.x); f[2] = bf16lo(r.y); f[3] = bf16hi(r.y);
     f[4] = bf16lo(r.z); f[5] = bf16hi(r.z); f[6] = bf16lo(r.w); f[7] = bf16hi(r.w);
-    if (p.silu) {
+    if (!GATED && p.silu) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) f[e] = silu_fast(f[e]);
       r = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
@@ -449,7 +600,7 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
     }
   };
   issue(0, 0);
-  __syncthreads();                              // pw is there
+  __syncthreads();                              // pw (gates, key sum) is there
   int st = 0;
   for (int t0 = 0; t0 < n_tok; t0 += CS_C, st ^= 1) {
     const int n = min(CS_C, n_tok - t0);
@@ -460,7 +611,7 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
     {
       float f[8];
 #pragma unroll 2
-      for (int i = 0; i < QP; ++i) {
+      for (int i = 0; !GATED && i < QP; ++i) {
         const int c = tid + i * CS_THREADS, t = c / (D / 8), d = (c % (D / 8)) * 8;
         silu_piece(Q + t * DS + d, f);
         silu_piece(K + t * DS + d, f);
@@ -469,7 +620,13 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
       for (int i = 0; i < VP; ++i) {
         const int c = tid + i * CS_THREADS, t = c / (CS_NV / 8), v = (c % (CS_NV / 8)) * 8;
         silu_piece(V + t * VS + v, f);
-        const float w = t < n ? pw[n - 1 - t] : 0.f;
+        float w = 0.f;
+        if constexpr (GATED) {
+          if (t < n) w = __expf(gts[st * 4 * CS_C + t] - tot[st * 2 + 1]);
+          if (v == 0) wgt[t] = w;
+        } else if (t < n) {
+          w = pw[n - 1 - t];
+        }
         uint4 hi, lo;
         split_bf16(f[0] * w, f[1] * w, hi.x, lo.x); split_bf16(f[2] * w, f[3] * w, hi.y, lo.y);
         split_bf16(f[4] * w, f[5] * w, hi.z, lo.z); split_bf16(f[6] * w, f[7] * w, hi.w, lo.w);
@@ -492,6 +649,42 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
     __syncthreads();
     if (t0 + CS_C < n_tok) issue(t0 + CS_C, st ^ 1);          // the other stage was last read before this barrier
     const int r0 = warp * 16 + gid, r1 = r0 + 8;              // this thread's two steps
+    const float* gt = gts + st * 4 * CS_C;
+    float nq0 = 0.f, nq1 = 0.f;                               // key sum before the chunk, times q, of the two steps
+    if constexpr (GATED) {
+      const float* ns = nsum + st * D;
+      const __nv_bfloat16* qr = Q + (warp * 16 + (lane >> 1)) * DS + (lane & 1) * (D / 2);
+      float s = 0.f;
+#pragma unroll 4
+      for (int d = 0; d < D / 2; d += 8) {
+        const uint4 r = *reinterpret_cast<const uint4*>(qr + d);
+        const float4 a = *reinterpret_cast<const float4*>(ns + (lane & 1) * (D / 2) + d), c = *reinterpret_cast<const float4*>(ns + (lane & 1) * (D / 2) + d + 4);
+        s += (bf16lo(r.x) * a.x + bf16hi(r.x) * a.y) + (bf16lo(r.y) * a.z + bf16hi(r.y) * a.w) +
+             (bf16lo(r.z) * c.x + bf16hi(r.z) * c.y) + (bf16lo(r.w) * c.z + bf16hi(r.w) * c.w);
+      }
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      nq0 = __shfl_sync(0xffffffffu, s, 2 * gid);
+      nq1 = __shfl_sync(0xffffffffu, s, 2 * gid + 16);
+      // key sum after the chunk, into the other stage
+      constexpr int PARTS = CS_THREADS / (D / 2);             // threads per pair of channels
+      const int d = tid / PARTS * 2, part = tid % PARTS;
+      float s0 = 0.f, s1 = 0.f;
+#pragma unroll 8
+      for (int t = part; t < CS_C; t += PARTS) {
+        const uint32_t r = *reinterpret_cast<const uint32_t*>(K + t * DS + d);
+        s0 += wgt[t] * bf16lo(r);
+        s1 += wgt[t] * bf16hi(r);
+      }
+#pragma unroll
+      for (int o = PARTS / 2; o > 0; o >>= 1) {
+        s0 += __shfl_xor_sync(0xffffffffu, s0, o);
+        s1 += __shfl_xor_sync(0xffffffffu, s1, o);
+      }
+      if (part == 0) {
+        nsum[(st ^ 1) * D + d] = tot[st * 2] * ns[d] + s0;
+        nsum[(st ^ 1) * D + d + 1] = tot[st * 2] * ns[d + 1] + s1;
+      }
+    }
     if (warp * 16 < n) {
       float o[CS_NV / 8][4], sc[CS_C / 8][4];
 #pragma unroll
@@ -519,7 +712,9 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
             mma_bf16_16816(sc[nt], qa, bb);
           }
       }
-      const float d0 = pw[r0 + 1], d1 = pw[r1 + 1];
+      const float d0 = GATED ? gt[2 * CS_C + r0] : pw[r0 + 1], d1 = GATED ? gt[2 * CS_C + r1] : pw[r1 + 1];
+      const float x0 = GATED ? gt[CS_C + r0] : 0.f, x1 = GATED ? gt[CS_C + r1] : 0.f;
+      float sum0 = 0.f, sum1 = 0.f;
 #pragma unroll
       for (int i = 0; i < CS_NV / 8; ++i) { o[i][0] *= d0; o[i][1] *= d0; o[i][2] *= d1; o[i][3] *= d1; }
 #pragma unroll
@@ -533,7 +728,12 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const int gap = (e < 2 ? r0 : r1) - (s + (e & 1));
-              f[e] = gap >= 0 ? sc[nt][e] * pw[gap] : 0.f;
+              if constexpr (GATED) f[e] = gap >= 0 ? sc[nt][e] * __expf(gt[s + (e & 1)] - (e < 2 ? x0 : x1)) : 0.f;
+              else f[e] = gap >= 0 ? sc[nt][e] * pw[gap] : 0.f;
+            }
+            if constexpr (GATED) {
+              sum0 += f[0] + f[1];
+              sum1 += f[2] + f[3];
             }
             split_bf16(f[0], f[1], ah[half * 2], al[half * 2]);
             split_bf16(f[2], f[3], ah[half * 2 + 1], al[half * 2 + 1]);
@@ -549,6 +749,17 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
             mma_bf16_16816(o[nv + 1], al, bb);
           }
         }
+      if constexpr (GATED) {
+#pragma unroll
+        for (int o = 1; o <= 2; o <<= 1) {
+          sum0 += __shfl_xor_sync(0xffffffffu, sum0, o);
+          sum1 += __shfl_xor_sync(0xffffffffu, sum1, o);
+        }
+        const float m0 = q_scale / (fmaxf(fabsf((d0 * nq0 + sum0) * q_scale), gt[3 * CS_C + r0]) + MLSTM_DEN_EPS);
+        const float m1 = q_scale / (fmaxf(fabsf((d1 * nq1 + sum1) * q_scale), gt[3 * CS_C + r1]) + MLSTM_DEN_EPS);
+#pragma unroll
+        for (int i = 0; i < CS_NV / 8; ++i) { o[i][0] *= m0; o[i][1] *= m0; o[i][2] *= m1; o[i][3] *= m1; }
+      }
       float* y = p.y + ((long long)b * p.T + t0) * p.nh * Dv + h * Dv + p0;
 #pragma unroll
       for (int nv = 0; nv < CS_NV / 8; ++nv) {
@@ -560,7 +771,7 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
       }
     }
     // state after the chunk
-    const float dn = pw[n];
+    const float dn = GATED ? tot[st * 2] : pw[n];
 #pragma unroll
     for (int mt = 0; mt < 2; ++mt)
 #pragma unroll
@@ -585,7 +796,14 @@ __global__ void __launch_bounds__(CS_THREADS, 2) decay_scan_chunk_kernel(LinearS
         }
       }
     }
+    if (GATED && warp == 0 && t0 + CS_C < n_tok) gates(t0 + CS_C, st ^ 1);
     __syncthreads();                            // the state and decayed-value copies are rewritten at the top of the next chunk
+  }
+  if constexpr (GATED) {
+    const int copies = min(CS_NV / MLSTM_SLICE, slices - sl0);
+    for (int i = tid; i < copies * D; i += CS_THREADS) p.key_sum[copy * D + i] = nsum[st * D + i % D];
+    if (tid == 0)
+      for (int c = 0; c < copies; ++c) p.run_max[copy + c] = m_run;
   }
 #pragma unroll
   for (int mt = 0; mt < 2; ++mt)
@@ -614,17 +832,17 @@ void opt_in(K kernel, size_t bytes) {
   if (bytes > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
 }
 
-template <typename T, bool DELTA>
+template <typename T, int KIND>
 void scan_go(const LinearScanParams& p, bool aligned, cudaStream_t st) {
   const dim3 grid((p.Dv + LS_PT - 1) / LS_PT, p.nh, p.B);
   auto go = [&](auto nj, auto al) {
     constexpr int NJ = decltype(nj)::value;
     constexpr bool AL = decltype(al)::value;
-    constexpr size_t stage = (DELTA ? 3 : 2) * LS_TT * NJ * 32 + LS_TT * LS_PT;
-    const size_t smem = sizeof(float) * (2 * stage + 2 * LS_TT + LS_TT * LS_PT);
-    auto kernel = linear_scan_kernel<T, DELTA, NJ, AL>;
+    constexpr size_t stage = (KIND == LS_DELTA ? 3 : 2) * LS_TT * NJ * 32 + LS_TT * LS_PT;
+    const size_t smem = sizeof(float) * (2 * stage + 2 * LS_TT + LS_TT * LS_PT + (KIND == LS_GATED ? 7 * LS_TT : 0));
+    auto kernel = linear_scan_kernel<T, KIND, NJ, AL>;
     opt_in(kernel, smem);
-    kernel<<<grid, LS_THREADS, smem, st>>>(p);
+    kernel<<<grid, LS_THREADS + (KIND == LS_GATED ? 32 : 0), smem, st>>>(p);
   };
   auto by_size = [&](auto al) {
     if (p.D <= 64) go(std::integral_constant<int, 2>{}, al);
@@ -633,6 +851,28 @@ void scan_go(const LinearScanParams& p, bool aligned, cudaStream_t st) {
   };
   if (aligned) by_size(std::true_type{}); else by_size(std::false_type{});
 }
+
+// prompt portions in bf16 whose sizes fit the chunked form; false: not launched
+template <bool GATED>
+bool chunk_go(const LinearScanParams& p, bool lp, cudaStream_t st) {
+  if (!lp || p.T < CS_MIN_T || (p.D != 64 && p.D != 128 && p.D != 256) || p.Dv % 8 != 0 || p.x_st % 8 != 0 || p.x_sb % 8 != 0 ||
+      (((uintptr_t)p.x | (uintptr_t)p.state | (uintptr_t)p.y) & 15) != 0)
+    return false;
+  const dim3 grid((p.Dv + CS_NV - 1) / CS_NV, p.nh, p.B);
+  auto go = [&](auto d) {
+    constexpr int D = decltype(d)::value;
+    const size_t smem = sizeof(__nv_bfloat16) * (2 * (2 * CS_C * (D + 8) + CS_C * (CS_NV + 8)) + 2 * CS_NV * (D + 8) + 2 * CS_C * (CS_NV + 8)) +
+                        sizeof(float) * (GATED ? 9 * CS_C + 4 + 2 * D : CS_C + 1);
+    opt_in(linear_chunk_kernel<D, GATED>, smem);
+    linear_chunk_kernel<D, GATED><<<grid, CS_THREADS, smem, st>>>(p);
+  };
+  if (p.D == 64) go(std::integral_constant<int, 64>{});
+  else if (p.D == 128) go(std::integral_constant<int, 128>{});
+  else go(std::integral_constant<int, 256>{});
+  return true;
+}
+
+static_assert(LS_PT == MLSTM_SLICE && CS_NV % MLSTM_SLICE == 0, "a block keeps whole copies of the key sum");
 
 }  // namespace
 
@@ -670,28 +910,23 @@ void channel_delta_scan_launch(const LinearScanParams& p, cudaStream_t st) {
   if (p.D > 256 || p.nh % p.n_qk != 0) throw std::runtime_error("channel_delta_scan: key size <= 256, heads a multiple of q / k heads");
   const bool aligned = p.D % 4 == 0 && p.Dv % 4 == 0 && p.x_st % 4 == 0 && p.x_sb % 4 == 0 &&
                        (((uintptr_t)p.x | (uintptr_t)p.decay | (uintptr_t)p.state) & 15) == 0;
-  scan_go<float, true>(p, aligned, st);
+  scan_go<float, LS_DELTA>(p, aligned, st);
 }
 
 void decay_scan_launch(const LinearScanParams& p, bool lp, cudaStream_t st) {
   if (p.B <= 0 || p.T <= 0) return;
   if (p.D > 256 || p.n_qk != p.nh) throw std::runtime_error("decay_scan: key size <= 256");
-  if (lp && p.T >= CS_MIN_T && (p.D == 64 || p.D == 128) && p.Dv % 8 == 0 && p.x_st % 8 == 0 && p.x_sb % 8 == 0 &&
-      (((uintptr_t)p.x | (uintptr_t)p.state | (uintptr_t)p.y) & 15) == 0) {
-    // prompt portions in bf16: chunks on tensor cores
-    const dim3 grid((p.Dv + CS_NV - 1) / CS_NV, p.nh, p.B);
-    auto go = [&](auto d) {
-      constexpr int D = decltype(d)::value;
-      const size_t smem = sizeof(__nv_bfloat16) * (2 * (2 * CS_C * (D + 8) + CS_C * (CS_NV + 8)) + 2 * CS_NV * (D + 8) + 2 * CS_C * (CS_NV + 8)) +
-                          sizeof(float) * (CS_C + 1);
-      opt_in(decay_scan_chunk_kernel<D>, smem);
-      decay_scan_chunk_kernel<D><<<grid, CS_THREADS, smem, st>>>(p);
-    };
-    if (p.D == 64) go(std::integral_constant<int, 64>{}); else go(std::integral_constant<int, 128>{});
-    return;
-  }
+  if (chunk_go<false>(p, lp, st)) return;
   const bool aligned = p.D % 4 == 0 && ((uintptr_t)p.state & 15) == 0;
-  if (lp) scan_go<__nv_bfloat16, false>(p, aligned, st); else scan_go<float, false>(p, aligned, st);
+  if (lp) scan_go<__nv_bfloat16, LS_FIXED>(p, aligned, st); else scan_go<float, LS_FIXED>(p, aligned, st);
+}
+
+void mlstm_scan_launch(const LinearScanParams& p, bool lp, cudaStream_t st) {
+  if (p.B <= 0 || p.T <= 0) return;
+  if (p.D > 256 || p.n_qk != p.nh) throw std::runtime_error("mlstm_scan: key size <= 256");
+  if (chunk_go<true>(p, lp, st)) return;
+  const bool aligned = p.D % 4 == 0 && ((uintptr_t)p.state & 15) == 0;
+  if (lp) scan_go<__nv_bfloat16, LS_GATED>(p, aligned, st); else scan_go<float, LS_GATED>(p, aligned, st);
 }
 
 void table_route_launch(const int* table, const int* ids, const int* q_len, float* w, int* idx, int B, int T, int k, int vocab, cudaStream_t st) {

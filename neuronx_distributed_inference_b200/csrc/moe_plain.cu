@@ -192,7 +192,7 @@ __global__ void __launch_bounds__(256) decode_down_kernel(const T* __restrict__ 
   if (lane == 0) stx(out + (size_t)tok * H + n, f);
 }
 
-// ---- fp32 router: logits, sigmoid scores, the k largest, renormalised ----------------------------------------------------------------
+// ---- fp32 router: logits (+ bias), scores, the k largest, renormalised ----------------------------------------------------------------
 // Kernel 1 (logits): block = RT tokens whose rows pass through shared memory as fp32, RKC columns at a time, x 8 warps; a warp forms the
 // logits of EG experts for all RT tokens from ONE pass over those experts' weight rows (RT x EG accumulators per lane: EG weight loads
 // and RT shared-memory loads feed RT * EG multiply-adds), so the router matrix is read once per RT tokens.  RT = 8 (sixteen tokens per block
@@ -280,7 +280,7 @@ __global__ void __launch_bounds__(256) router_logits_kernel(const T* __restrict_
     }
 }
 
-__global__ void __launch_bounds__(256) router_select_kernel(const float* __restrict__ logits, float* __restrict__ topk_w, int* __restrict__ topk_i,
+__global__ void __launch_bounds__(256) router_select_kernel(float* __restrict__ logits, float* __restrict__ topk_w, int* __restrict__ topk_i,
                                                             int N, int E, int k, RouterSelect sel) {
   extern __shared__ float zsm[];                             // per warp: [E] scores, [E] choice scores, [groups] group bests
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -290,11 +290,21 @@ __global__ void __launch_bounds__(256) router_select_kernel(const float* __restr
   float* sc = zsm + (size_t)warp * (2 * E + G);
   float* ch = sc + E;
   float* gb = ch + E;
-  // scores: sigmoid, or softmax over all router outputs
+  // scores: sigmoid, softmax over all router outputs, or the logits themselves (softmax over the chosen ones at the end)
   float mx = -INFINITY;
-  for (int e = lane; e < E; e += 32) { const float v = logits[(size_t)tok * E + e]; sc[e] = v; mx = fmaxf(mx, v); }
-  if (sel.softmax) {
-    mx = warp_max(mx);
+  for (int e = lane; e < E; e += 32) {
+    float v = logits[(size_t)tok * E + e];
+    if (sel.bias) {
+      v += sel.bias[e];
+      logits[(size_t)tok * E + e] = v;
+    }
+    sc[e] = v;
+    mx = fmaxf(mx, v);
+  }
+  mx = warp_max(mx);
+  if (sel.softmax == 2) {
+    // nothing to do: the choice goes by the logits
+  } else if (sel.softmax) {
     float den = 0.f;
     for (int e = lane; e < E; e += 32) { const float v = expf(sc[e] - mx); sc[e] = v; den += v; }
     den = warp_sum(den);
@@ -345,7 +355,7 @@ __global__ void __launch_bounds__(256) router_select_kernel(const float* __restr
     float best;
     int bi;
     arg_max(ch, E, best, bi);
-    const float w = sc[bi];
+    const float w = sel.softmax == 2 ? expf(sc[bi] - mx) : sc[bi];
     sum += w;
     if (lane == 0) {
       topk_w[(size_t)tok * k + j] = w;
@@ -354,7 +364,7 @@ __global__ void __launch_bounds__(256) router_select_kernel(const float* __restr
     }
     __syncwarp();
   }
-  const float mul = (sel.renorm_eps >= 0.f ? 1.f / (sum + sel.renorm_eps) : 1.f) * sel.scale;
+  const float mul = (sel.softmax == 2 ? 1.f / sum : sel.renorm_eps >= 0.f ? 1.f / (sum + sel.renorm_eps) : 1.f) * sel.scale;
   if (mul != 1.f)
     for (int j = lane; j < k; j += 32) topk_w[(size_t)tok * k + j] *= mul;
 }

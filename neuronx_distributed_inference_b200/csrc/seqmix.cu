@@ -115,11 +115,15 @@ __global__ void __launch_bounds__(256) conv_qknorm_rope_append_kernel(ConvQkPara
   const int Cq = p.n_q * p.D, Ck = p.n_kv * p.D, Cv = p.n_kv * p.Dv, C = Cq + Ck + Cv, K = p.K;
   const bool has_ctx = p.ctx_len[b] > 0;
   const T* u0 = (const T*)p.p + (long long)b * p.p_sb;
-  const T* sl = (const T*)p.state + (long long)p.lines[b] * (K - 1) * C;
+  const T* sl = K > 1 ? (const T*)p.state + (long long)p.lines[b] * (K - 1) * C : nullptr;
   float sq = 0.f, sk = 0.f;
   for (int c = threadIdx.x; c < C; c += blockDim.x) {
     float acc = 0.f;
-    for (int j = 0; j < K; ++j) acc += p.conv_w[(long long)c * K + j] * conv_input(u0, p.p_st, sl, C, K, t - K + 1 + j, c, has_ctx);
+    if (p.conv_w) {
+      for (int j = 0; j < K; ++j) acc += p.conv_w[(long long)c * K + j] * conv_input(u0, p.p_st, sl, C, K, t - K + 1 + j, c, has_ctx);
+    } else {
+      acc = ldf(u0 + (long long)t * p.p_st + c);
+    }
     buf[c] = acc;
     if (c < Cq) sq += acc * acc;
     else if (c < Cq + Ck) sk += acc * acc;
@@ -146,9 +150,11 @@ __global__ void __launch_bounds__(256) conv_qknorm_rope_append_kernel(ConvQkPara
     const int d = cc % p.D;
     float self = buf[c] * r * (nw ? nw[cc] : 1.f);
     if (d < p.R) {
-      const float other = buf[c ^ 1] * r * (nw ? nw[cc ^ 1] : 1.f);
-      const float co = cs[d >> 1], si = sn[d >> 1];
-      self = (d & 1) ? (self * co + other * si) : (self * co - other * si);
+      const int hr = p.R / 2;
+      const bool second = p.half ? d >= hr : (d & 1);
+      const int step = (p.half ? hr : 1) * (second ? -1 : 1), i = p.half ? (second ? d - hr : d) : d >> 1;
+      const float other = buf[c + step] * r * (nw ? nw[cc + step] : 1.f);
+      self = second ? (self * cs[i] + other * sn[i]) : (self * cs[i] - other * sn[i]);
     }
     stf((isq ? qo : ko) + cc, self);
   }
@@ -176,17 +182,23 @@ __global__ void __launch_bounds__(256) conv_qknorm_rope_append_pair_kernel(ConvQ
   const int Cq = p.n_q * p.D, Ck = p.n_kv * p.D, Cv = p.n_kv * p.Dv, C = Cq + Ck + Cv, K = p.K;
   const bool has_ctx = p.ctx_len[b] > 0;
   const T* u0 = (const T*)p.p + (long long)b * p.p_sb;
-  const T* sl = (const T*)p.state + (long long)p.lines[b] * (K - 1) * C;
+  const T* sl = K > 1 ? (const T*)p.state + (long long)p.lines[b] * (K - 1) * C : nullptr;
   float sq = 0.f, sk = 0.f;
   for (int c = 2 * threadIdx.x; c < C; c += 2 * blockDim.x) {
     float a0 = 0.f, a1 = 0.f;
-    for (int j = 0; j < K; ++j) {
-      const int i = t - K + 1 + j;
-      float2 v = make_float2(0.f, 0.f);
-      if (i >= 0) v = ld2(u0 + (long long)i * p.p_st + c);
-      else if (has_ctx) v = ld2(sl + (long long)(K - 1 + i) * C + c);
-      a0 += p.conv_w[(long long)c * K + j] * v.x;
-      a1 += p.conv_w[(long long)(c + 1) * K + j] * v.y;
+    if (p.conv_w) {
+      for (int j = 0; j < K; ++j) {
+        const int i = t - K + 1 + j;
+        float2 v = make_float2(0.f, 0.f);
+        if (i >= 0) v = ld2(u0 + (long long)i * p.p_st + c);
+        else if (has_ctx) v = ld2(sl + (long long)(K - 1 + i) * C + c);
+        a0 += p.conv_w[(long long)c * K + j] * v.x;
+        a1 += p.conv_w[(long long)(c + 1) * K + j] * v.y;
+      }
+    } else {
+      const float2 v = ld2(u0 + (long long)t * p.p_st + c);
+      a0 = v.x;
+      a1 = v.y;
     }
     buf[c] = a0;
     buf[c + 1] = a1;
@@ -215,7 +227,19 @@ __global__ void __launch_bounds__(256) conv_qknorm_rope_append_pair_kernel(ConvQ
     const float* nw = isq ? p.q_norm_w : p.k_norm_w;
     const int d = cc % p.D;
     float a = buf[c] * r * (nw ? nw[cc] : 1.f), bb = buf[c + 1] * r * (nw ? nw[cc + 1] : 1.f);
-    if (d < p.R) {
+    if (p.half) {
+      // channel i pairs with i + R / 2: the partners come from the row in shared memory (R / 2 may be odd: each channel on its own)
+      const int hr = p.R / 2;
+      auto turn = [&](float self, int o) {
+        if (d + o >= p.R) return self;
+        const bool second = d + o >= hr;
+        const int step = second ? -hr : hr, i = second ? d + o - hr : d + o;
+        const float other = buf[c + o + step] * r * (nw ? nw[cc + o + step] : 1.f);
+        return second ? self * cs[i] + other * sn[i] : self * cs[i] - other * sn[i];
+      };
+      a = turn(a, 0);
+      bb = turn(bb, 1);
+    } else if (d < p.R) {
       const float co = cs[d >> 1], si = sn[d >> 1];
       const float ra = a * co - bb * si, rb = bb * co + a * si;
       a = ra;
@@ -925,6 +949,41 @@ template <> __device__ __forceinline__ void st4<__nv_bfloat16>(__nv_bfloat16* p,
   *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
 }
 
+// out = rms_unit(alpha * x + y) * (offset + w), the sums in registers between the two passes (rows up to NCH * 1024 wide)
+template <typename TY, int NCH>
+__global__ void __launch_bounds__(256) scaled_add_rmsnorm_vec_kernel(const float* __restrict__ x, const TY* __restrict__ y,
+                                                                     const float* __restrict__ w, float* __restrict__ out,
+                                                                     __nv_bfloat16* __restrict__ out_lp, int W, float alpha, float eps,
+                                                                     float offset) {
+  __shared__ float red[32];
+  const long long row = (long long)blockIdx.x * W;
+  float4 s[NCH];
+  float ss = 0.f;
+#pragma unroll
+  for (int ch = 0; ch < NCH; ++ch) {
+    const int c = (ch * 256 + threadIdx.x) * 4;
+    s[ch] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c >= W) continue;
+    const float4 v = ld4(x + row + c), a = y ? ld4(y + row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    s[ch] = make_float4(alpha * v.x + a.x, alpha * v.y + a.y, alpha * v.z + a.z, alpha * v.w + a.w);
+    ss += s[ch].x * s[ch].x + s[ch].y * s[ch].y + s[ch].z * s[ch].z + s[ch].w * s[ch].w;
+  }
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)W + eps);
+#pragma unroll
+  for (int ch = 0; ch < NCH; ++ch) {
+    const int c = (ch * 256 + threadIdx.x) * 4;
+    if (c >= W) continue;
+    float4 g = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (w) {
+      g = ld4(w + c);
+      g = make_float4(g.x + offset, g.y + offset, g.z + offset, g.w + offset);
+    }
+    const float4 o = make_float4(s[ch].x * r * g.x, s[ch].y * r * g.y, s[ch].z * r * g.z, s[ch].w * r * g.w);
+    st4(out + row + c, o);
+    if (out_lp) st4(out_lp + row + c, o);
+  }
+}
+
 template <typename TY, typename TH, int NCH>
 __global__ void __launch_bounds__(256) stream_add_rmsnorm_vec_kernel(StreamAddParams p) {
   __shared__ float red[32];
@@ -988,7 +1047,7 @@ __global__ void __launch_bounds__(256) latent_norm_append_kernel(const T* __rest
                                                                  int page, int max_blocks, float eps, T* __restrict__ rows_out, int rot,
                                                                  const float* __restrict__ cosv, const float* __restrict__ sinv,
                                                                  const T* __restrict__ q_in, int q_rank, const float* __restrict__ q_w,
-                                                                 T* __restrict__ q_out) {
+                                                                 T* __restrict__ q_out, int interleaved) {
   const int lane = threadIdx.x & 31;
   const long long tok = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   if (tok >= (long long)B * Tn) return;
@@ -1017,13 +1076,14 @@ __global__ void __launch_bounds__(256) latent_norm_append_kernel(const T* __rest
   const int RW = R + rot;                                 // cache row: the latent, then the rotated key part
   T* dst = cache + ((long long)block_table[(long long)b * max_blocks + pos / page] * page + pos % page) * RW;
   T* dst2 = rows_out ? rows_out + tok * RW : nullptr;     // [B, T, RW]: the same rows in token order
-  for (int i = lane; i < rot / 2; i += 32) {              // rotate-half: channel i pairs with i + rot / 2
-    const float u = ldf(row + R + i), v = ldf(row + R + rot / 2 + i);
+  for (int i = lane; i < rot / 2; i += 32) {              // channel i pairs with i + rot / 2, or 2i with 2i + 1
+    const int c0 = interleaved ? 2 * i : i, c1 = interleaved ? 2 * i + 1 : rot / 2 + i;
+    const float u = ldf(row + R + c0), v = ldf(row + R + c1);
     const float co = cosv[tok * (rot / 2) + i], si = sinv[tok * (rot / 2) + i];
     const float a = u * co - v * si, bb = v * co + u * si;
-    stf(dst + R + i, a);
-    stf(dst + R + rot / 2 + i, bb);
-    if (dst2) { stf(dst2 + R + i, a); stf(dst2 + R + rot / 2 + i, bb); }
+    stf(dst + R + c0, a);
+    stf(dst + R + c1, bb);
+    if (dst2) { stf(dst2 + R + c0, a); stf(dst2 + R + c1, bb); }
   }
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
@@ -1041,20 +1101,22 @@ __global__ void __launch_bounds__(256) latent_norm_append_kernel(const T* __rest
   }
 }
 
-// dst[tok, h, Dd - rot + .] = rotate_half(src[tok, h, Ds - rot + .]); one thread per (token, head, pair)
+// dst[tok, h, Dd - rot + .] = rotate(src[tok, h, Ds - rot + .]); one thread per (token, head, pair)
 template <typename T>
-__global__ void __launch_bounds__(256) rope_half_tail_kernel(const T* __restrict__ src, T* __restrict__ dst, const float* __restrict__ cosv,
-                                                             const float* __restrict__ sinv, long long n, int H, int Ds, int Dd, int rot) {
+__global__ void __launch_bounds__(256) rope_tail_kernel(const T* __restrict__ src, T* __restrict__ dst, const float* __restrict__ cosv,
+                                                             const float* __restrict__ sinv, long long n, int H, int Ds, int Dd, int rot,
+                                                             int interleaved) {
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= n) return;
   const int half = rot / 2, i = (int)(idx % half);
   const long long th = idx / half, tok = th / H;
   const T* sr = src + th * Ds + (Ds - rot);
   T* dr = dst + th * Dd + (Dd - rot);
-  const float u = ldf(sr + i), v = ldf(sr + half + i);
+  const int c0 = interleaved ? 2 * i : i, c1 = interleaved ? 2 * i + 1 : half + i;
+  const float u = ldf(sr + c0), v = ldf(sr + c1);
   const float co = cosv[tok * half + i], si = sinv[tok * half + i];
-  stf(dr + i, u * co - v * si);
-  stf(dr + half + i, v * co + u * si);
+  stf(dr + c0, u * co - v * si);
+  stf(dr + c1, v * co + u * si);
 }
 
 // Stream update + norm + short convolution of the normalised rows.  Block = one token; window row j (j < K) is the stream row at
@@ -2063,9 +2125,9 @@ __global__ void __launch_bounds__(DL2_THREADS) gated_delta_scan_wide_kernel(Delt
     }
 }
 
-// ---- per-head RMS norm with a shared weight, times an activated gate: one warp per (row, head) ------------------------------------------
+// ---- per-head RMS norm (weight shared by the heads or one per channel), times an activated gate: one warp per (row, head) ------------------------------------------
 template <typename TG, typename TO>
-__global__ void __launch_bounds__(128) head_rmsnorm_gate_kernel(const float* __restrict__ y, const float* __restrict__ w, const TG* __restrict__ gate,
+__global__ void __launch_bounds__(128) head_rmsnorm_gate_kernel(const float* __restrict__ y, const float* __restrict__ w, int w_stride, const TG* __restrict__ gate,
                                                                 long long g_stride, TO* __restrict__ out, long long nrh, int H, int Dv, float eps,
                                                                 int act) {
   const long long i = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -2073,6 +2135,7 @@ __global__ void __launch_bounds__(128) head_rmsnorm_gate_kernel(const float* __r
   const int lane = threadIdx.x & 31, h = (int)(i % H);
   const long long row = i / H;
   const float* yr = y + i * Dv;
+  w += (long long)h * w_stride;
   float v[SEQMIX_MAX_VDIM / 32], ss = 0.f;
 #pragma unroll
   for (int k = 0; k < SEQMIX_MAX_VDIM / 32; ++k) {
@@ -2100,6 +2163,20 @@ void opt_in_smem(K kernel, size_t bytes) {
 void scaled_add_rmsnorm_launch(const float* x, const void* y, bool y_lp, const float* w, float* out, void* out_lp, int rows, int W,
                                float alpha, float eps, float offset, cudaStream_t st) {
   if (rows <= 0) return;
+  auto al = [](const void* q, size_t a) { return ((uintptr_t)q & (a - 1)) == 0; };
+  if (W % 4 == 0 && W >= 256 && W <= 8192 && al(x, 16) && al(y, y_lp ? 8 : 16) && al(w, 16) && al(out, 16) && al(out_lp, 8)) {
+    const int nch = (W + 1023) / 1024;
+    auto go = [&](auto tag) {
+      using TY = decltype(tag);
+      auto run = [&](auto kernel) { kernel<<<rows, 256, 0, st>>>(x, (const TY*)y, w, out, (__nv_bfloat16*)out_lp, W, alpha, eps, offset); };
+      if (nch <= 1) run(scaled_add_rmsnorm_vec_kernel<TY, 1>);
+      else if (nch <= 2) run(scaled_add_rmsnorm_vec_kernel<TY, 2>);
+      else if (nch <= 4) run(scaled_add_rmsnorm_vec_kernel<TY, 4>);
+      else run(scaled_add_rmsnorm_vec_kernel<TY, 8>);
+    };
+    if (y_lp) go(__nv_bfloat16{}); else go(float{});
+    return;
+  }
   if (y_lp)
     scaled_add_rmsnorm_kernel<__nv_bfloat16><<<rows, 256, 0, st>>>(x, (const __nv_bfloat16*)y, w, out, (__nv_bfloat16*)out_lp, W, alpha, eps, offset);
   else
@@ -2139,26 +2216,26 @@ void stream_add_rmsnorm_launch(const StreamAddParams& p, bool y_lp, bool h_lp, c
 void latent_norm_append_launch(const void* p, long long p_sb, long long p_st, const float* w, void* cache, const int* block_table,
                                const int* ctx_len, const int* q_len, int B, int T, int R, int page, int max_blocks, float eps, bool lp,
                                void* rows_out, int rot, const float* cos, const float* sin, const void* q_in, int q_rank, const float* q_w,
-                               void* q_out, cudaStream_t st) {
+                               void* q_out, bool interleaved, cudaStream_t st) {
   if (B <= 0 || T <= 0) return;
   const unsigned grid = (unsigned)(((long long)B * T + 7) / 8);
   if (lp)
     latent_norm_append_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>((const __nv_bfloat16*)p, p_sb, p_st, w, (__nv_bfloat16*)cache, block_table, ctx_len,
                                                                    q_len, B, T, R, page, max_blocks, eps, (__nv_bfloat16*)rows_out, rot, cos, sin,
-                                                                   (const __nv_bfloat16*)q_in, q_rank, q_w, (__nv_bfloat16*)q_out);
+                                                                   (const __nv_bfloat16*)q_in, q_rank, q_w, (__nv_bfloat16*)q_out, (int)interleaved);
   else
     latent_norm_append_kernel<float><<<grid, 256, 0, st>>>((const float*)p, p_sb, p_st, w, (float*)cache, block_table, ctx_len, q_len, B, T, R, page,
                                                            max_blocks, eps, (float*)rows_out, rot, cos, sin, (const float*)q_in, q_rank, q_w,
-                                                           (float*)q_out);
+                                                           (float*)q_out, (int)interleaved);
 }
 
-void rope_half_tail_launch(const void* src, void* dst, const float* cos, const float* sin, long long tokens, int H, int Ds, int Dd, int rot, bool lp,
-                           cudaStream_t st) {
+void rope_tail_launch(const void* src, void* dst, const float* cos, const float* sin, long long tokens, int H, int Ds, int Dd, int rot,
+                      bool interleaved, bool lp, cudaStream_t st) {
   const long long n = tokens * H * (rot / 2);
   if (n <= 0) return;
   const unsigned grid = (unsigned)((n + 255) / 256);
-  if (lp) rope_half_tail_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>((const __nv_bfloat16*)src, (__nv_bfloat16*)dst, cos, sin, n, H, Ds, Dd, rot);
-  else rope_half_tail_kernel<float><<<grid, 256, 0, st>>>((const float*)src, (float*)dst, cos, sin, n, H, Ds, Dd, rot);
+  if (lp) rope_tail_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>((const __nv_bfloat16*)src, (__nv_bfloat16*)dst, cos, sin, n, H, Ds, Dd, rot, (int)interleaved);
+  else rope_tail_kernel<float><<<grid, 256, 0, st>>>((const float*)src, (float*)dst, cos, sin, n, H, Ds, Dd, rot, (int)interleaved);
 }
 
 void stream_norm_conv_launch(const StreamConvParams& p, bool out_lp, cudaStream_t st) {
@@ -2461,17 +2538,17 @@ void gated_delta_scan_launch(const DeltaScanParams& p, bool lp, cudaStream_t st)
   }
 }
 
-void head_rmsnorm_gate_launch(const float* y, const float* w, const void* gate, long long g_stride, void* out, long long rows, int H, int Dv,
+void head_rmsnorm_gate_launch(const float* y, const float* w, int w_stride, const void* gate, long long g_stride, void* out, long long rows, int H, int Dv,
                               float eps, int act, bool gate_lp, bool out_lp, cudaStream_t st) {
   const long long nrh = rows * H;
   if (nrh <= 0) return;
   const unsigned grid = (unsigned)((nrh + 3) / 4);
   if (gate_lp) {
-    if (out_lp) head_rmsnorm_gate_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, 128, 0, st>>>(y, w, (const __nv_bfloat16*)gate, g_stride, (__nv_bfloat16*)out, nrh, H, Dv, eps, act);
-    else head_rmsnorm_gate_kernel<__nv_bfloat16, float><<<grid, 128, 0, st>>>(y, w, (const __nv_bfloat16*)gate, g_stride, (float*)out, nrh, H, Dv, eps, act);
+    if (out_lp) head_rmsnorm_gate_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, 128, 0, st>>>(y, w, w_stride, (const __nv_bfloat16*)gate, g_stride, (__nv_bfloat16*)out, nrh, H, Dv, eps, act);
+    else head_rmsnorm_gate_kernel<__nv_bfloat16, float><<<grid, 128, 0, st>>>(y, w, w_stride, (const __nv_bfloat16*)gate, g_stride, (float*)out, nrh, H, Dv, eps, act);
   } else {
-    if (out_lp) head_rmsnorm_gate_kernel<float, __nv_bfloat16><<<grid, 128, 0, st>>>(y, w, (const float*)gate, g_stride, (__nv_bfloat16*)out, nrh, H, Dv, eps, act);
-    else head_rmsnorm_gate_kernel<float, float><<<grid, 128, 0, st>>>(y, w, (const float*)gate, g_stride, (float*)out, nrh, H, Dv, eps, act);
+    if (out_lp) head_rmsnorm_gate_kernel<float, __nv_bfloat16><<<grid, 128, 0, st>>>(y, w, w_stride, (const float*)gate, g_stride, (__nv_bfloat16*)out, nrh, H, Dv, eps, act);
+    else head_rmsnorm_gate_kernel<float, float><<<grid, 128, 0, st>>>(y, w, w_stride, (const float*)gate, g_stride, (float*)out, nrh, H, Dv, eps, act);
   }
 }
 

@@ -30,16 +30,16 @@ struct StreamAddParams {
 void stream_add_rmsnorm_launch(const StreamAddParams& p, bool y_lp, bool h_lp, cudaStream_t st);
 
 // p points at the latent slice of the projection rows.  rot > 0: the `rot` channels behind the latent are rotated (rotate-half
-// layout, cos / sin [B, T, rot / 2]) and stored behind the latent in the cache row of R + rot numbers.  q_rank > 0: channels
+// layout, or pairs (2i, 2i + 1) when interleaved; cos / sin [B, T, rot / 2]) and stored behind the latent in the cache row of R + rot numbers.  q_rank > 0: channels
 // [0, q_rank) of the rows at `q_in` (same strides) are RMS-normalised with q_w into q_out [B, T, q_rank].
 void latent_norm_append_launch(const void* p, long long p_sb, long long p_st, const float* w, void* cache, const int* block_table,
                                const int* ctx_len, const int* q_len, int B, int T, int R, int page, int max_blocks, float eps, bool lp,
                                void* rows_out, int rot, const float* cos, const float* sin, const void* q_in, int q_rank, const float* q_w,
-                               void* q_out, cudaStream_t st);      // rows_out: [B, T, R + rot] copy of the live rows in token order, or null
+                               void* q_out, bool interleaved, cudaStream_t st);      // rows_out: [B, T, R + rot] copy of the live rows in token order, or null
 
-// dst[b, t, h, Dd - rot ...] = rotate_half(src[b, t, h, Ds - rot ...]) with cos / sin [B * T, rot / 2]
-void rope_half_tail_launch(const void* src, void* dst, const float* cos, const float* sin, long long tokens, int H, int Ds, int Dd, int rot, bool lp,
-                           cudaStream_t st);
+// dst[b, t, h, Dd - rot ...] = rotate(src[b, t, h, Ds - rot ...]) with cos / sin [B * T, rot / 2]; pairs as in latent_norm_append
+void rope_tail_launch(const void* src, void* dst, const float* cos, const float* sin, long long tokens, int H, int Ds, int Dd, int rot,
+                      bool interleaved, bool lp, cudaStream_t st);
 
 // s = x + [y1] + [y2]; h = rms_unit(s) * w; out = h + sum_j cw[:, j] * h_(t - K + 1 + j), the rows before a portion from the fp32 state
 // line (stream rows, normalised like the new ones; zero when ctx_len == 0).  cw null: out = h.
@@ -83,10 +83,11 @@ void moe_plain_gate_mul_launch(const void* gu, void* h, int R, int I, int act, f
                                cudaStream_t st);
 
 // fp32 router: logits = x W^T (x bf16 or fp32, W fp32 [E, W]) on CUDA cores with the rows in shared memory, then per token the
-// scores (sigmoid, or softmax over all E) of the k experts with the largest score + correction among the `keep` best of `groups` equal
+// scores (sigmoid, softmax over all E, or softmax over the chosen logits) of the k experts with the largest score + correction among the `keep` best of `groups` equal
 // groups of neighbours, divided by their sum + renorm_eps when renorm_eps >= 0, times scale.  `logits` [N, E] is written and read.
 struct RouterSelect {
-  int softmax;               // 0: sigmoid scores
+  int softmax;               // 0: sigmoid scores, 1: softmax over all outputs, 2: the largest logits, softmax over them alone
+  const float* bias;         // [E] or null: added to the logits
   const float* correction;   // [E] or null: added to the scores for the choice only
   int groups, keep;          // groups <= 1: no group limit
   float renorm_eps, scale;
@@ -104,8 +105,8 @@ void short_conv_update_launch(const void* u, long long u_sb, long long u_st, voi
 struct ConvQkParams {
   const void* p;            // [B, T, >= Cq + Ck + Cv] projections, row strides below
   long long p_sb, p_st;
-  const float* conv_w;      // [Cq + Ck + Cv, K]
-  const void* state;        // [lines, K - 1, Cq + Ck + Cv]
+  const float* conv_w;      // [Cq + Ck + Cv, K] or null (no convolution, K = 1)
+  const void* state;        // [lines, K - 1, Cq + Ck + Cv] or null (K = 1)
   const int *lines, *ctx_len, *q_len;
   const float *q_norm_w, *k_norm_w;
   const float *cos, *sin;   // [B, T, R / 2]
@@ -113,6 +114,7 @@ struct ConvQkParams {
   void *k_cache, *v_cache;  // [blocks, page, n_kv, D | Dv]
   const int* block_table;   // [B, max_blocks]
   int B, T, K, n_q, n_kv, D, Dv, R, page, max_blocks;
+  int half;                 // rotation pairs (i, i + R / 2) instead of (2i, 2i + 1)
   float eps;
 };
 void conv_qknorm_rope_append_launch(const ConvQkParams& p, bool lp, cudaStream_t st);
@@ -202,8 +204,9 @@ struct DeltaScanParams {
 };
 void gated_delta_scan_launch(const DeltaScanParams& p, bool lp, cudaStream_t st);
 
-// out[row, h, :] = rms_unit(y[row, h, :]) * w[:] * act(gate[row, h, :]); w [Dv] is shared by the heads; gate rows g_stride elements apart
-void head_rmsnorm_gate_launch(const float* y, const float* w, const void* gate, long long g_stride, void* out, long long rows, int H, int Dv,
+// out[row, h, :] = rms_unit(y[row, h, :]) * w[h * w_stride + :] * act(gate[row, h, :]); w_stride 0: weight [Dv] shared by the heads, Dv: one
+// per channel; gate rows g_stride elements apart
+void head_rmsnorm_gate_launch(const float* y, const float* w, int w_stride, const void* gate, long long g_stride, void* out, long long rows, int H, int Dv,
                               float eps, int act, bool gate_lp, bool out_lp, cudaStream_t st);
 
 // gate non-null: times act(gate) after the norm; gate rows g_stride elements apart
@@ -258,9 +261,36 @@ struct LinearScanParams {
   const int *lines, *ctx_len, *q_len;
   float* y;                        // [B, T, nh Dv]
   int B, T, nh, n_qk, D, Dv, silu; // silu: SiLU on q, k and v as they are read (fixed decays only)
+  // exponential input gates only
+  int gate_at;                     // channel of the raw input gates (then the forget gates) in a row
+  const float *i_bias, *f_bias;    // [nh]
+  float cap;
+  float *key_sum, *run_max;        // [lines, nh, slices, D], [lines, nh, slices]: one copy per MLSTM_SLICE value channels
 };
+constexpr int MLSTM_SLICE = 16;
 void channel_delta_scan_launch(const LinearScanParams& p, cudaStream_t st);
 void decay_scan_launch(const LinearScanParams& p, bool lp, cudaStream_t st);
+
+// Matrix memory with exponential input gates (linear_scan.cu).  Rows q | k | v | .. with the raw input and forget gates (one per head each) at
+// channel gate_at; per head i = cap tanh((raw + i_bias) / cap), f = logsigmoid(cap tanh((raw + f_bias) / cap)), m' = max(f + m, i),
+// S' = exp(f + m - m') S + exp(i - m') v k^T, n' likewise with k alone, y = S' q / (max(|n' q|, exp(-m')) + 1e-6), q scaled by D^-1/2.
+// n and m are kept once per MLSTM_SLICE value channels, so that no block reads what another block of the launch writes.
+void mlstm_scan_launch(const LinearScanParams& p, bool lp, cudaStream_t st);
+
+// x[tok] = embed[id] * scale + bigram[(prev * mul_prev + id * mul_cur) mod buckets] (row `buckets` for a sequence's first token), fp32 and
+// optionally bf16; prev of a portion's first token comes from the sequence's line, which then takes the portion's last token
+struct BigramEmbedParams {
+  const int* ids;                  // [B, T]
+  const void *embed, *bigram;      // [vocab, W], [buckets + 1, W] or null
+  int* state;                      // [lines, 1] or null (no bigram)
+  const int *lines, *ctx_len, *q_len;
+  float* x;                        // [B, T, W]
+  void* x_lp;                      // bf16 copy or null
+  long long mul_prev, mul_cur, buckets;
+  int B, T, W, vocab;
+  float scale;
+};
+void bigram_embed_launch(const BigramEmbedParams& p, bool lp, cudaStream_t st);
 
 // idx[i, j] = table[ids[i], j] (-1 for tokens past q_len), w[i, j] = 1 / k
 void table_route_launch(const int* table, const int* ids, const int* q_len, float* w, int* idx, int B, int T, int k, int vocab, cudaStream_t st);

@@ -88,18 +88,20 @@ void short_conv_update(const at::Tensor& u, at::Tensor state, const at::Tensor& 
                            qlen.data_ptr<int>(), (int)B, (int)u.size(1), (int)C, (int)K, is_lp(u), stream());
 }
 
-at::Tensor conv_qknorm_rope_append(const at::Tensor& p, const at::Tensor& conv_w, const at::Tensor& state, const at::Tensor& lines,
+at::Tensor conv_qknorm_rope_append(const at::Tensor& p, const OptT& conv_w, const OptT& state, const at::Tensor& lines,
                                    const at::Tensor& ctx, const at::Tensor& qlen, const OptT& q_norm_w, const OptT& k_norm_w, double eps,
                                    int64_t n_q, int64_t n_kv, int64_t D, int64_t Dv, const OptT& cos, const OptT& sin,
-                                   at::Tensor k_cache, at::Tensor v_cache, const OptT& block_table) {
+                                   at::Tensor k_cache, at::Tensor v_cache, const OptT& block_table, bool half) {
   check_act(p, "conv_qknorm_rope_append projections");
   check_rows(p, "conv_qknorm_rope_append projections");
-  const int64_t B = p.size(0), T = p.size(1), C = n_q * D + n_kv * (D + Dv), K = conv_w.size(1);
+  const int64_t B = p.size(0), T = p.size(1), C = n_q * D + n_kv * (D + Dv), K = conv_w.has_value() ? conv_w->size(1) : 1;
   TORCH_CHECK(p.size(2) >= C && D % 2 == 0, "conv_qknorm_rope_append: projection narrower than q | k | v, or odd head size");
-  check_f32(conv_w, "conv weight");
-  TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(0) == C && K >= 1 && K <= SEQMIX_MAX_TAPS);
-  TORCH_CHECK(state.is_cuda() && state.scalar_type() == p.scalar_type() && state.is_contiguous() && state.dim() == 3 &&
-              state.size(1) == K - 1 && state.size(2) == C, "conv_qknorm_rope_append: state [lines, taps - 1, q | k | v channels]");
+  if (conv_w.has_value()) {
+    check_f32(*conv_w, "conv weight");
+    TORCH_CHECK(conv_w->dim() == 2 && conv_w->size(0) == C && K >= 1 && K <= SEQMIX_MAX_TAPS);
+  }
+  TORCH_CHECK(K == 1 || (state.has_value() && state->is_cuda() && state->scalar_type() == p.scalar_type() && state->is_contiguous() && state->dim() == 3 &&
+              state->size(1) == K - 1 && state->size(2) == C), "conv_qknorm_rope_append: state [lines, taps - 1, q | k | v channels]");
   check_i32(lines, B, "lines");
   check_i32(ctx, B, "ctx_len");
   check_i32(qlen, B, "q_len");
@@ -139,7 +141,7 @@ at::Tensor conv_qknorm_rope_append(const at::Tensor& p, const at::Tensor& conv_w
   c10::cuda::CUDAGuard guard(p.device());
   auto q = at::zeros({B, T, n_q, D}, p.options());
   a.p = p.data_ptr(); a.p_sb = p.stride(0); a.p_st = p.stride(1);
-  a.conv_w = conv_w.data_ptr<float>(); a.state = state.data_ptr();
+  a.conv_w = conv_w.has_value() ? conv_w->data_ptr<float>() : nullptr; a.state = K > 1 ? state->data_ptr() : nullptr; a.half = half ? 1 : 0;
   a.lines = lines.data_ptr<int>(); a.ctx_len = ctx.data_ptr<int>(); a.q_len = qlen.data_ptr<int>();
   a.q_norm_w = q_norm_w.has_value() ? q_norm_w->data_ptr<float>() : nullptr;
   a.cos = cos.has_value() ? cos->data_ptr<float>() : nullptr;
@@ -395,6 +397,61 @@ at::Tensor decay_scan(const at::Tensor& x, const at::Tensor& decay, at::Tensor s
   return y;
 }
 
+at::Tensor mlstm_scan(const at::Tensor& x, int64_t gate_at, const at::Tensor& i_bias, const at::Tensor& f_bias, double cap, at::Tensor state,
+                      at::Tensor key_sum, at::Tensor run_max, const at::Tensor& lines, const at::Tensor& ctx, const at::Tensor& qlen, int64_t nh,
+                      int64_t D, int64_t Dv) {
+  check_act(x, "mlstm_scan rows");
+  check_rows(x, "mlstm_scan rows");
+  check_f32(i_bias, "mlstm_scan input gate bias"); check_f32(f_bias, "mlstm_scan forget gate bias");
+  check_f32(state, "mlstm_scan state"); check_f32(key_sum, "mlstm_scan key sum"); check_f32(run_max, "mlstm_scan running maximum");
+  const int64_t B = x.size(0), T = x.size(1), NS = (Dv + MLSTM_SLICE - 1) / MLSTM_SLICE;
+  TORCH_CHECK(gate_at >= nh * (2 * D + Dv) && x.size(2) >= gate_at + 2 * nh && i_bias.numel() == nh && f_bias.numel() == nh && D >= 1 && D <= 256 && cap > 0,
+              "mlstm_scan: rows q | k | v .. input gates | forget gates, one bias per head, key size <= 256, positive cap");
+  TORCH_CHECK(state.dim() == 4 && state.size(1) == nh && state.size(2) == Dv && state.size(3) == D, "mlstm_scan: state [lines, heads, Dv, D]");
+  TORCH_CHECK(key_sum.dim() == 4 && key_sum.size(0) == state.size(0) && key_sum.size(1) == nh && key_sum.size(2) == NS && key_sum.size(3) == D,
+              "mlstm_scan: key sum [lines, heads, slices, D]");
+  TORCH_CHECK(run_max.dim() == 3 && run_max.size(0) == state.size(0) && run_max.size(1) == nh && run_max.size(2) == NS,
+              "mlstm_scan: running maximum [lines, heads, slices]");
+  check_i32(lines, B, "lines"); check_i32(ctx, B, "ctx_len"); check_i32(qlen, B, "q_len");
+  c10::cuda::CUDAGuard guard(x.device());
+  auto y = at::zeros({B, T, nh * Dv}, x.options().dtype(at::kFloat));
+  LinearScanParams p{};
+  p.x = x.data_ptr(); p.x_sb = x.stride(0); p.x_st = x.stride(1); p.gate_at = (int)gate_at;
+  p.i_bias = i_bias.data_ptr<float>(); p.f_bias = f_bias.data_ptr<float>(); p.cap = (float)cap;
+  p.state = state.data_ptr<float>(); p.key_sum = key_sum.data_ptr<float>(); p.run_max = run_max.data_ptr<float>();
+  p.lines = lines.data_ptr<int>(); p.ctx_len = ctx.data_ptr<int>(); p.q_len = qlen.data_ptr<int>(); p.y = y.data_ptr<float>();
+  p.B = (int)B; p.T = (int)T; p.nh = p.n_qk = (int)nh; p.D = (int)D; p.Dv = (int)Dv;
+  mlstm_scan_launch(p, is_lp(x), stream());
+  return y;
+}
+
+std::tuple<at::Tensor, OptT> bigram_embed(const at::Tensor& ids, const at::Tensor& embed, const OptT& bigram, double scale, int64_t mul_prev,
+                                          int64_t mul_cur, const OptT& state, const at::Tensor& lines, const at::Tensor& ctx, const at::Tensor& qlen,
+                                          bool want_lp) {
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kInt && ids.dim() == 2 && ids.is_contiguous(), "bigram_embed: ids [B, T] int32");
+  check_act(embed, "bigram_embed table");
+  TORCH_CHECK(embed.dim() == 2 && embed.is_contiguous());
+  const int64_t B = ids.size(0), T = ids.size(1), W = embed.size(1);
+  check_i32(lines, B, "lines"); check_i32(ctx, B, "ctx_len"); check_i32(qlen, B, "q_len");
+  BigramEmbedParams p{};
+  if (bigram.has_value()) {
+    TORCH_CHECK(bigram->is_cuda() && bigram->scalar_type() == embed.scalar_type() && bigram->is_contiguous() && bigram->dim() == 2 &&
+                bigram->size(0) >= 2 && bigram->size(1) == W && mul_prev >= 0 && mul_cur >= 0, "bigram_embed: bigram table [buckets + 1, W]");
+    TORCH_CHECK(state.has_value() && state->is_cuda() && state->scalar_type() == at::kInt && state->is_contiguous() && state->dim() == 2 &&
+                state->size(1) == 1, "bigram_embed: state [lines, 1] int32");
+    p.bigram = bigram->data_ptr(); p.state = state->data_ptr<int>(); p.buckets = bigram->size(0) - 1;
+  }
+  c10::cuda::CUDAGuard guard(ids.device());
+  auto x = at::empty({B, T, W}, embed.options().dtype(at::kFloat));
+  OptT lp;
+  if (want_lp) lp = at::empty({B, T, W}, embed.options().dtype(at::kBFloat16));
+  p.ids = ids.data_ptr<int>(); p.embed = embed.data_ptr(); p.lines = lines.data_ptr<int>(); p.ctx_len = ctx.data_ptr<int>();
+  p.q_len = qlen.data_ptr<int>(); p.x = x.data_ptr<float>(); p.x_lp = lp.has_value() ? lp->data_ptr() : nullptr;
+  p.mul_prev = mul_prev; p.mul_cur = mul_cur; p.B = (int)B; p.T = (int)T; p.W = (int)W; p.vocab = (int)embed.size(0); p.scale = (float)scale;
+  bigram_embed_launch(p, is_lp(embed), stream());
+  return {x, lp};
+}
+
 std::tuple<at::Tensor, at::Tensor> table_route(const at::Tensor& table, const at::Tensor& ids, const at::Tensor& qlen) {
   TORCH_CHECK(table.is_cuda() && table.scalar_type() == at::kInt && table.is_contiguous() && table.dim() == 2, "table_route: table [vocab, k] int32");
   TORCH_CHECK(ids.dim() == 2);
@@ -481,7 +538,7 @@ std::tuple<at::Tensor, OptT, OptT> stream_add_rmsnorm(const OptT& x, const OptT&
 
 std::tuple<OptT, OptT> latent_norm_append(const at::Tensor& p, int64_t offset, int64_t rank, const at::Tensor& w, double eps, at::Tensor cache,
                                           const at::Tensor& block_table, const at::Tensor& ctx, const at::Tensor& qlen, bool emit_rows, int64_t rot,
-                                          const OptT& cos, const OptT& sin, int64_t q_rank, const OptT& q_w) {
+                                          const OptT& cos, const OptT& sin, int64_t q_rank, const OptT& q_w, bool interleaved) {
   check_act(p, "latent_norm_append input");
   check_rows(p, "latent_norm_append input");
   const int64_t B = p.size(0), T = p.size(1);
@@ -514,7 +571,7 @@ std::tuple<OptT, OptT> latent_norm_append(const at::Tensor& p, int64_t offset, i
                             qlen.data_ptr<int>(), (int)B, (int)T, (int)rank, (int)cache.size(1), (int)block_table.size(1), (float)eps, is_lp(p),
                             rows.has_value() ? rows->data_ptr() : nullptr, (int)rot, rot > 0 ? cos->data_ptr<float>() : nullptr,
                             rot > 0 ? sin->data_ptr<float>() : nullptr, p.data_ptr(), (int)q_rank, q_rank > 0 ? q_w->data_ptr<float>() : nullptr,
-                            cq.has_value() ? cq->data_ptr() : nullptr, stream());
+                            cq.has_value() ? cq->data_ptr() : nullptr, interleaved, stream());
   return {rows, cq};
 }
 
@@ -606,8 +663,8 @@ at::Tensor moe_plain(const at::Tensor& x, const at::Tensor& w_up, const at::Tens
   return out;
 }
 
-std::tuple<at::Tensor, at::Tensor, at::Tensor> router_topk(const at::Tensor& x, const at::Tensor& w, int64_t k, double renorm_eps, bool softmax,
-                                                           const OptT& correction, int64_t groups, int64_t keep, double scale) {
+std::tuple<at::Tensor, at::Tensor, at::Tensor> router_topk(const at::Tensor& x, const at::Tensor& w, const OptT& bias, int64_t k, double renorm_eps,
+                                                           int64_t softmax, const OptT& correction, int64_t groups, int64_t keep, double scale) {
   check_act(x, "router input");
   check_f32(w, "router weight");
   TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && w.dim() == 2 && w.size(1) == x.size(1) && k >= 1 && k <= w.size(0));
@@ -618,7 +675,13 @@ std::tuple<at::Tensor, at::Tensor, at::Tensor> router_topk(const at::Tensor& x, 
   auto tw = at::empty({N, k}, f32);
   auto ti = at::empty({N, k}, x.options().dtype(at::kInt));
   RouterSelect sel{};
-  sel.softmax = softmax ? 1 : 0;
+  TORCH_CHECK(softmax >= 0 && softmax <= 2);
+  sel.softmax = (int)softmax;
+  if (bias.has_value()) {
+    check_f32(*bias, "router bias");
+    TORCH_CHECK(bias->numel() == E);
+    sel.bias = bias->data_ptr<float>();
+  }
   if (correction.has_value()) {
     check_f32(*correction, "router score correction");
     TORCH_CHECK(correction->numel() == E);
@@ -630,18 +693,18 @@ std::tuple<at::Tensor, at::Tensor, at::Tensor> router_topk(const at::Tensor& x, 
   return {logits, tw, ti};
 }
 
-void rope_half_tail(const at::Tensor& src, at::Tensor dst, int64_t rot, const at::Tensor& cos, const at::Tensor& sin) {
-  check_act(src, "rope_half_tail source");
+void rope_tail(const at::Tensor& src, at::Tensor dst, int64_t rot, const at::Tensor& cos, const at::Tensor& sin, bool interleaved) {
+  check_act(src, "rope_tail source");
   TORCH_CHECK(src.dim() == 4 && dst.dim() == 4 && src.is_contiguous() && dst.is_contiguous() && dst.is_cuda() && dst.scalar_type() == src.scalar_type() &&
               src.size(0) == dst.size(0) && src.size(1) == dst.size(1) && src.size(2) == dst.size(2) && rot % 2 == 0 && rot <= src.size(3) &&
-              rot <= dst.size(3), "rope_half_tail: [B, T, H, D] tensors of one type");
+              rot <= dst.size(3), "rope_tail: [B, T, H, D] tensors of one type");
   check_f32(cos, "cos");
   check_f32(sin, "sin");
   const int64_t tokens = src.size(0) * src.size(1);
   TORCH_CHECK(cos.numel() == tokens * (rot / 2) && sin.numel() == cos.numel(), "cos / sin [B, T, rot / 2]");
   c10::cuda::CUDAGuard guard(src.device());
-  rope_half_tail_launch(src.data_ptr(), dst.data_ptr(), cos.data_ptr<float>(), sin.data_ptr<float>(), tokens, (int)src.size(2), (int)src.size(3),
-                        (int)dst.size(3), (int)rot, is_lp(src), stream());
+  rope_tail_launch(src.data_ptr(), dst.data_ptr(), cos.data_ptr<float>(), sin.data_ptr<float>(), tokens, (int)src.size(2), (int)src.size(3),
+                   (int)dst.size(3), (int)rot, interleaved, is_lp(src), stream());
 }
 
 std::tuple<at::Tensor, at::Tensor> stream_norm_conv(const at::Tensor& x, const OptT& y1, const OptT& y2, const at::Tensor& w, const OptT& cw,
@@ -817,12 +880,13 @@ at::Tensor head_rmsnorm_gate(const at::Tensor& y, const at::Tensor& w, int64_t h
   check_f32(w, "head_rmsnorm_gate weight");
   TORCH_CHECK(y.dim() == 2 && y.size(1) % heads == 0);
   const int64_t rows = y.size(0), Dv = y.size(1) / heads;
-  TORCH_CHECK(w.numel() == Dv && Dv <= SEQMIX_MAX_VDIM, "head_rmsnorm_gate: weight [Dv], Dv <= ", SEQMIX_MAX_VDIM);
+  TORCH_CHECK((w.numel() == Dv || w.numel() == y.size(1)) && Dv <= SEQMIX_MAX_VDIM, "head_rmsnorm_gate: weight [Dv] or [heads * Dv], Dv <= ",
+              SEQMIX_MAX_VDIM);
   check_act(gate, "head_rmsnorm_gate gate");
   TORCH_CHECK(gate.dim() == 2 && gate.size(0) == rows && gate.size(1) == y.size(1) && gate.stride(1) == 1, "head_rmsnorm_gate: gate [rows, heads * Dv]");
   c10::cuda::CUDAGuard guard(y.device());
   auto out = at::empty(y.sizes(), y.options().dtype(out_lp ? at::kBFloat16 : at::kFloat));
-  head_rmsnorm_gate_launch(y.data_ptr<float>(), w.data_ptr<float>(), gate.data_ptr(), gate.stride(0), out.data_ptr(), rows, (int)heads, (int)Dv,
+  head_rmsnorm_gate_launch(y.data_ptr<float>(), w.data_ptr<float>(), w.numel() == Dv ? 0 : (int)Dv, gate.data_ptr(), gate.stride(0), out.data_ptr(), rows, (int)heads, (int)Dv,
                            (float)eps, (int)act, is_lp(gate), out_lp, stream());
   return out;
 }
@@ -838,9 +902,11 @@ void register_seqmix(pybind11::module_& m) {
   m.def("delta_front", &delta_front);
   m.def("channel_delta_scan", &channel_delta_scan);
   m.def("decay_scan", &decay_scan);
+  m.def("mlstm_scan", &mlstm_scan);
+  m.def("bigram_embed", &bigram_embed);
   m.def("table_route", &table_route);
   m.def("router_topk", &router_topk);
-  m.def("rope_half_tail", &rope_half_tail);
+  m.def("rope_tail", &rope_tail);
   m.def("stream_norm_conv", &stream_norm_conv);
   m.def("identity_expert_add", &identity_expert_add);
   m.def("stream_add_rmsnorm", &stream_add_rmsnorm);

@@ -77,6 +77,7 @@ class FetodraInferenceConfig(InferenceConfig):
 
 
 class NeuronFetodraModel(NeuronBaseModel):
+    design = "Fetodra"
     meta_extra_keys = ("computed_context_lens",)
     # decode steps (one token per row) replay from a CUDA graph: these per-step tensors are staged into the graph's static inputs
     graph_tensor_kwargs = ("slot_mapping", "block_table", "computed_context_lens", "gather_positions")
@@ -90,9 +91,9 @@ class NeuronFetodraModel(NeuronBaseModel):
     def setup_attr_for_model(self, config):
         nc = config.neuron_config
         if nc.tp_degree != 1:
-            raise NotImplementedError("Fetodra: tensor parallel degree 1 (row-wide q/k norms and the grouped scan are not sharded)")
+            raise NotImplementedError(f"{self.design}: tensor parallel degree 1 (row-wide q/k norms and the grouped scan are not sharded)")
         if not nc.is_block_kv_layout:
-            raise ValueError("Fetodra runs on the paged KV cache: set is_block_kv_layout=True, pa_block_size, pa_num_blocks")
+            raise ValueError(f"{self.design} runs on the paged KV cache: set is_block_kv_layout=True, pa_block_size, pa_num_blocks")
         self.tp_degree, self.hidden_size = 1, config.width
         self.max_batch_size, self.buckets = nc.max_batch_size, nc.buckets
 
@@ -148,7 +149,7 @@ class NeuronFetodraModel(NeuronBaseModel):
     def build_meta(self, input_ids, attention_mask, position_ids, seq_ids, is_prefill, **kw):
         meta = super().build_meta(input_ids, attention_mask, position_ids, seq_ids, is_prefill, **kw)
         if meta.block_table is None:
-            raise ValueError("Fetodra: every forward needs block_table (paged KV cache)")
+            raise ValueError(f"{self.design}: every forward needs block_table (paged KV cache)")
         B, T = input_ids.shape[:2]
         dev = input_ids.device
         q_len = meta.key_valid.sum(-1).to(torch.int32) if meta.key_valid is not None else torch.full((B,), T, dtype=torch.int32, device=dev)

@@ -439,6 +439,10 @@ class NeuronBaseModel(nn.Module):
         return self.tp_group.size > 1 and not getattr(self.lm_head, "gather_output", True)
 
     # ------------------------------------------------------------------------------------
+    def embed_step(self, input_ids, meta: AttnMeta, inputs_embeds=None, vision_embeddings=None, vision_mask=None):
+        """Embedding of one forward's tokens; models whose embedding reads per-sequence state (an earlier token) override this."""
+        return self.embed(input_ids, inputs_embeds, vision_embeddings, vision_mask)
+
     def embed(self, input_ids, inputs_embeds=None, vision_embeddings=None, vision_mask=None):
         h = inputs_embeds if inputs_embeds is not None else self.embed_tokens(input_ids)
         if vision_embeddings is not None and vision_mask is not None:
@@ -504,7 +508,7 @@ class NeuronBaseModel(nn.Module):
         meta = self.build_meta(input_ids, attention_mask, position_ids, seq_ids, is_prefill, **kw)
         if self.tp_group.symm is not None:
             self.tp_group.symm.begin_step()     # fresh tags for this forward's in-kernel collectives (parallel/symm.py)
-        h = self.embed(input_ids, inputs_embeds, vision_embeddings, vision_mask)
+        h = self.embed_step(input_ids, meta, inputs_embeds, vision_embeddings, vision_mask)
         sp = self._set_sequence_parallel(is_prefill and T % self.tp_group.size == 0 and T >= self.tp_group.size)
         if sp:
             # sequence parallel prefill (reference model_base.py:1471-1583): the residual stream is sharded along the

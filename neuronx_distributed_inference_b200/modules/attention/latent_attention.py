@@ -11,7 +11,8 @@ no positional rotations.  Constructor parameters, so that other stacks can combi
 * ``scale``: multiplies the scores;
 * ``q_rank``: queries pass a latent of their own, ``q = W_uq rms_norm(W_dq x)``, instead of one projection;
 * ``rot_dim`` / ``rope``: every query head carries ``rot_dim`` extra channels and every token ONE extra key part of ``rot_dim`` channels
-  shared by all heads; both are rotated by position (rotate-half layout; ``rope = (inv_freq fp64, magnitude, tag)``) and their product
+  shared by all heads; both are rotated by position (rotate-half layout, or pairs ``(2i, 2i+1)`` with ``rope_interleaved``;
+  ``rope = (inv_freq fp64, magnitude, tag)``) and their product
   joins the score.  The rotated key part is stored behind the latent in the same cache row, so a row is ``kv_rank + rot_dim`` numbers,
   the key of the multi-query attention is the whole row and its value the first ``kv_rank`` numbers;
 * ``window``: position ``i`` sees ``j`` iff ``0 <= i - j < window``;
@@ -22,7 +23,7 @@ Data flow (CUDA: csrc/seqmix.cu for the two middle steps, GEMMs around them):
 
     p   = W_in x                          q (or its latent) | latent | rotated key part | gates in ONE GEMM
           latent_norm_append(p)           fp32 RMS norm of the latent slice(s), rotation of the shared key part, paged cache write
-    a   = q_h U_h                         batched over heads (rotated query channels appended by rope_half_tail)
+    a   = q_h U_h                         batched over heads (rotated query channels appended by rope_tail)
     l   = paged_window_attention(a)       fp32 softmax (+ sink) over the latent cache, times sigmoid(gate_h)
     y   = W_o [V_h l_h]                   batched over heads, then the output projection
 
@@ -41,7 +42,7 @@ from .conv_window_attention import ragged_rope_tables
 class LatentSinkAttention(nn.Module):
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, kv_rank: int, *, scale: float, eps: float,
                  sink: bool = True, head_gate: bool = True, layer_idx: int = 0, dtype=torch.bfloat16, device=None, tp_group=None,
-                 q_rank: int = 0, rot_dim: int = 0, rope=None, window=None, channel_gate: bool = False):
+                 q_rank: int = 0, rot_dim: int = 0, rope=None, window=None, channel_gate: bool = False, rope_interleaved: bool = False):
         super().__init__()
         if tp_group is not None and tp_group.size != 1:
             raise NotImplementedError("latent attention: the latent row is shared by all heads; tensor parallel degree 1")
@@ -50,8 +51,9 @@ class LatentSinkAttention(nn.Module):
         self.n_q, self.head_dim, self.v_head_dim, self.kv_rank = num_heads, head_dim, v_head_dim, kv_rank
         self.scale, self.eps, self.layer_idx = float(scale), float(eps), layer_idx
         self.q_rank, self.rot_dim, self.window, self.channel_gate = int(q_rank or 0), int(rot_dim or 0), (int(window) if window else None), channel_gate
-        # the first slice of the input projection: the queries themselves, or their latent
-        self.Cq = self.q_rank or num_heads * head_dim
+        self.interleaved = bool(rope_interleaved)
+        # the first slice of the input projection: the queries themselves (per head: unrotated, then rotated channels), or their latent
+        self.Cq = self.q_rank or num_heads * (head_dim + self.rot_dim)
         self.Cg = num_heads * v_head_dim if channel_gate else (num_heads if head_gate else 0)
         self.in_proj = ColumnParallelLinear(hidden_size, self.Cq + kv_rank + self.rot_dim + self.Cg, bias=False, gather_output=False, dtype=dtype,
                                             device=device, tensor_model_parallel_group=tp_group)
@@ -87,17 +89,18 @@ class LatentSinkAttention(nn.Module):
         whole = (meta.is_prefill and not meta.has_prefix and T >= 16 and not rot and not self.window
                  and ops.latent_prefill_on_tensor_cores(p, R))
         rows = ops.latent_norm_append(p, self.Cq, R, self.latent_norm_weight, self.eps, cache, meta.block_table, ctx, qlen, emit_rows=whole,
-                                      rot_dim=rot, cos=cos, sin=sin, q_rank=self.q_rank, q_weight=self.q_norm_weight if self.q_rank else None)
+                                      rot_dim=rot, cos=cos, sin=sin, q_rank=self.q_rank, q_weight=self.q_norm_weight if self.q_rank else None,
+                                      interleaved=self.interleaved)
         if self.q_rank:
             rows, cq = rows
             q = self.q_up(cq).view(B * T, H, d + rot)
         else:
-            q = p.view(B * T, -1)[:, :self.Cq].unflatten(1, (H, d))
+            q = p.view(B * T, -1)[:, :self.Cq].unflatten(1, (H, d + rot))
         # batched over heads with strided operands and results: the products land in [B, T, H, .] layout, no transposing copies
         a = torch.empty(B, T, H, R + rot, dtype=p.dtype, device=p.device)
         torch.bmm(q[..., :d].transpose(0, 1), self.k_up, out=a.view(B * T, H, R + rot)[..., :R].transpose(0, 1))
         if rot:
-            ops.rope_half_tail(q.view(B, T, H, d + rot), a, rot, cos, sin)
+            ops.rope_tail(q.view(B, T, H, d + rot), a, rot, cos, sin, self.interleaved)
         gate = p[..., self.Cq + R + rot:] if self.Cg else None
         head_gate = gate if not self.channel_gate else None
         if whole:

@@ -1,5 +1,6 @@
 """Recurrent mixers on ragged rows with carried state (chunked prompts, mixed prefill / decode batches): Mamba-2, the gated delta rule (one
-decay per head, or one per head and key channel) and linear attention with a fixed decay per head.
+decay per head, or one per head and key channel), linear attention with a fixed decay per head and the matrix memory with exponential
+input gates (mLSTM).
 
 ``in_proj`` rows are ``[z: inner | x: inner | B: G N | C: G N | dt: heads]``.  x, B and C pass a depthwise causal convolution (+bias)
 and SiLU; ``dt = softplus(dt + dt_bias)``; per head ``S <- exp(-exp(A_log) dt) S + dt B x^T`` (fp32, ``[N, head_dim]``),
@@ -216,3 +217,60 @@ class RaggedDecayMixer(nn.Module):
                            self.D, self.Dv, True)
         y = ops.group_rmsnorm(y, self.norm_weight, 1, self.eps, out_dtype=p.dtype, gate=p[..., self.qkv:], act="sigmoid")
         return self.out_proj(y)
+
+
+class RaggedMatrixMemoryMixer(nn.Module):
+    """Matrix memory with exponential input gates (mLSTM) on ragged rows.  Projection rows are ``[q: heads D | k: heads D | v: heads Dv | out
+    gate: heads Dv | input gate: heads | forget gate: heads]`` in one GEMM (padded with zero rows to a multiple of 8).  Both gates are
+    capped, ``cap tanh(. / cap)`` after their bias; the memory ``S [Dv, D]``, the key sum ``n`` and the running maximum ``m`` of a head follow
+    ``m' = max(f + m, i)``, ``S' = e^(f + m - m') S + e^(i - m') v k^T``, ``n'`` likewise with ``k`` alone, and the output is
+    ``S' q / (max(|n' . q|, e^-m') + 1e-6)`` with ``q`` scaled by ``D^-1/2``.  Every head is divided by its root mean square, the concatenation
+    multiplied by a weight per channel and by ``sigmoid`` of the out gate, and projected out.  Gates, memory, key sum, maximum and norm are
+    fp32 whatever the activation dtype; all of them start at zero and live in the sequence's state line.  CUDA: csrc/linear_scan.cu
+    (mlstm_scan: recurrent form, and a chunked form on tensor cores for bf16 portions), csrc/seqmix.cu (head_rmsnorm_gate)."""
+
+    def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, gate_cap: float, eps: float, layer_idx: int,
+                 dtype=torch.bfloat16, device=None, tp_group=None):
+        super().__init__()
+        if tp_group is not None and tp_group.size != 1:
+            raise NotImplementedError("ragged matrix-memory mixer: tensor parallel degree 1")
+        self.nh, self.D, self.Dv, self.cap, self.eps, self.layer_idx = num_heads, head_dim, v_head_dim, float(gate_cap), eps, layer_idx
+        self.inner, self.qkv = num_heads * v_head_dim, num_heads * (2 * head_dim + v_head_dim)
+        self.in_width = -(-(self.qkv + self.inner + 2 * num_heads) // 8) * 8
+        self.in_proj = ColumnParallelLinear(hidden_size, self.in_width, bias=False, gather_output=False, dtype=dtype, device=device,
+                                            tensor_model_parallel_group=tp_group)
+        self.out_proj = RowParallelLinear(self.inner, hidden_size, bias=False, input_is_parallel=True, dtype=dtype, device=device,
+                                          tensor_model_parallel_group=tp_group)
+        f32 = dict(dtype=torch.float32, device=device)
+        self.i_bias = nn.Parameter(torch.zeros(num_heads, **f32), requires_grad=False)
+        self.f_bias = nn.Parameter(torch.zeros(num_heads, **f32), requires_grad=False)
+        self.norm_weight = nn.Parameter(torch.ones(self.inner, **f32), requires_grad=False)
+
+    @staticmethod
+    def stack(*parts):
+        """The projections in the order of ``in_proj``'s rows, zero rows behind them up to a multiple of 8."""
+        w = torch.cat(parts, 0)
+        return torch.cat([w, w.new_zeros(-w.shape[0] % 8, w.shape[1])], 0)
+
+    def _names(self, run):
+        run = self.layer_idx if run is None else run
+        return tuple(f"matrix_memory_{part}.run{run}" for part in ("state", "keys", "max"))
+
+    def state_specs(self, cache_index=None):
+        state, keys, top = self._names(cache_index)
+        slices = -(-self.Dv // ops.MLSTM_SLICE)
+        return {state: ((self.nh, self.Dv, self.D), torch.float32), keys: ((self.nh, slices, self.D), torch.float32),
+                top: ((self.nh, slices), torch.float32)}
+
+    def forward(self, x, meta, kv_mgr, cache_index=None):
+        ex = meta.extras
+        p = self.in_proj(x)
+        C = self.qkv + self.inner
+        o = ops.mlstm_scan(p, C, self.i_bias, self.f_bias, self.cap, *(kv_mgr.states.tensor(n) for n in self._names(cache_index)),
+                           ex["state_lines"], ex["ctx_len"], ex["q_len"], self.nh, self.D, self.Dv)
+        gate = p[..., self.qkv:C]
+        if self.Dv <= 256:
+            o = ops.head_rmsnorm_gate(o, self.norm_weight, self.nh, self.eps, gate, "sigmoid", out_dtype=p.dtype)
+        else:
+            o = ops.group_rmsnorm(o, self.norm_weight, self.nh, self.eps, out_dtype=p.dtype, gate=gate, act="sigmoid")
+        return self.out_proj(o)

@@ -63,6 +63,7 @@ def rmsnorm(x, weight, eps: float, offset: float = 0.0, residual=None):
     return ref.rmsnorm(x, weight, eps, offset, residual)
 
 
+_GATE_PRODUCTS = {"silu_mul": "silu", "gelu_tanh_mul": "gelu_tanh", "gelu_mul": "gelu"}
 _ACT_CODES = {None: 0, "silu_mul": 1, "gelu_tanh_mul": 2, "gelu_mul": 3}
 
 
@@ -128,12 +129,12 @@ def linear(x, w, bias=None, norm_weight=None, norm_eps: float = 1e-6, norm_offse
                 y = _C().gemm(x2.contiguous(), w, bias, _ACT_CODES[act], r2, o2)
                 y = out if out is not None else y.view(*x.shape[:-1], y.shape[-1])
                 return y if (residual is None or r2 is not None) else y + residual
-    if act == "silu_mul" and _mix_cuda(x) and w.dtype == x.dtype and scale is None and x.dim() >= 2:
+    if act in _GATE_PRODUCTS and _mix_cuda(x) and w.dtype == x.dtype and scale is None and x.dim() >= 2:
         # fp32 rows and sizes the GEMM kernels do not take: library product, then the gate product as one elementwise kernel
         gu = ref.linear(x, w, bias, norm_weight, norm_eps, norm_offset)
         g2 = gu.reshape(-1, gu.shape[-1])
         n = g2.shape[-1] // 2
-        y = gated_act_mul(g2[:, :n], g2[:, n:], "silu").view(*gu.shape[:-1], n)
+        y = gated_act_mul(g2[:, :n], g2[:, n:], _GATE_PRODUCTS[act]).view(*gu.shape[:-1], n)
     else:
         y = ref.linear(x, w, bias, norm_weight, norm_eps, norm_offset, act, scale)
     y = y if residual is None else y + residual
@@ -358,20 +359,21 @@ def moe_route(router_logits, top_k, act="softmax", normalize=True, act_over_topk
 
 
 def router_topk(x, weight, top_k, act="softmax", normalize=True, act_over_topk=False, renorm_eps=None, correction=None, groups=None,
-                scale=1.0):
-    """fp32 router: ``logits = x W^T`` (W fp32), then :func:`moe_route`.  Sigmoid routers, and softmax routers that are not
-    renormalised or that choose by corrected scores among kept groups, run as two kernels on CUDA (fp32 products with the rows in
+                scale=1.0, bias=None):
+    """fp32 router: ``logits = x W^T + bias`` (W, bias fp32), then :func:`moe_route`.  Sigmoid routers, softmax routers that are not
+    renormalised or that choose by corrected scores among kept groups, and softmax over the chosen logits alone (``act_over_topk``) run as two kernels on CUDA (fp32 products with the rows in
     shared memory; scores, group limit, selection and scaling, one warp per token) instead of a cast, a library GEMM and a chain of
     elementwise / sort launches.  -> (logits, weights [N, k] fp32, expert ids [N, k])."""
     E = weight.shape[0]
     plain_softmax = act == "softmax" and (not normalize or correction is not None or groups is not None)
-    if (_mix_cuda(x) and (act == "sigmoid" or plain_softmax) and not act_over_topk and weight.dtype == torch.float32 and x.dim() == 2
-            and top_k <= E and E <= 512 and (groups is None or (E % int(groups[0]) == 0 and int(groups[1]) <= int(groups[0])))):
+    over_topk = act == "softmax" and act_over_topk and correction is None and groups is None and renorm_eps is None and scale == 1.0
+    if (_mix_cuda(x) and (over_topk or ((act == "sigmoid" or plain_softmax) and not act_over_topk)) and weight.dtype == torch.float32
+            and x.dim() == 2 and (bias is None or bias.dtype == torch.float32) and top_k <= E and E <= 512 and (groups is None or (E % int(groups[0]) == 0 and int(groups[1]) <= int(groups[0])))):
         stats["router_topk"] += 1
         count, keep = (int(groups[0]), int(groups[1])) if groups is not None else (1, 1)
-        return _C().router_topk(x.contiguous(), weight.contiguous(), int(top_k), -1.0 if renorm_eps is None else float(renorm_eps),
-                                act == "softmax", None if correction is None else correction.float().contiguous(), count, keep, float(scale))
-    logits = torch.nn.functional.linear(x.float(), weight.float())
+        return _C().router_topk(x.contiguous(), weight.contiguous(), None if bias is None else bias.contiguous(), int(top_k),
+                                -1.0 if renorm_eps is None else float(renorm_eps), 2 if over_topk else int(act == "softmax"), None if correction is None else correction.float().contiguous(), count, keep, float(scale))
+    logits = torch.nn.functional.linear(x.float(), weight.float(), None if bias is None else bias.float())
     w, idx = moe_route(logits, top_k, act, normalize, act_over_topk, renorm_eps, correction, groups, scale)
     return logits, w, idx
 
@@ -524,15 +526,16 @@ def short_conv_update(u, state, slots, ctx_len, q_len):
 
 
 def conv_qknorm_rope_append(qkv, conv_w, state, slots, ctx_len, q_len, q_norm_w, k_norm_w, eps, n_q, n_kv, D, Dv, cos, sin,
-                            k_cache, v_cache, block_table, out_dtype=None):
-    if _mix_cuda(qkv) and qkv.stride(-1) == 1 and conv_w.shape[1] <= _MIX_MAX_TAPS and D % 2 == 0:
+                            k_cache, v_cache, block_table, out_dtype=None, half: bool = False):
+    """``conv_w = None``: no convolution; ``half``: rotation pairs (i, i + R/2) instead of (2i, 2i+1) (definition: ops/reference.py)."""
+    if _mix_cuda(qkv) and qkv.stride(-1) == 1 and (conv_w is None or conv_w.shape[1] <= _MIX_MAX_TAPS) and D % 2 == 0:
         stats["conv_qknorm_rope_append"] += 1
         return _C().conv_qknorm_rope_append(qkv, conv_w, state, _i32(slots), _i32(ctx_len), _i32(q_len), q_norm_w, k_norm_w, float(eps),
                                             int(n_q), int(n_kv), int(D), int(Dv), None if cos is None else cos.float().contiguous(),
                                             None if sin is None else sin.float().contiguous(),
-                                            k_cache, v_cache, None if block_table is None else _i32(block_table))
+                                            k_cache, v_cache, None if block_table is None else _i32(block_table), bool(half))
     return ref.conv_qknorm_rope_append(qkv, conv_w, state, slots, ctx_len, q_len, q_norm_w, k_norm_w, eps, n_q, n_kv, D, Dv, cos, sin,
-                                       k_cache, v_cache, block_table, out_dtype)
+                                       k_cache, v_cache, block_table, out_dtype, half)
 
 
 def paged_window_attention(q, k_cache, v_cache, block_table, ctx_len, q_len, scale, softcap, window, keep_first, gate=None, sinks=None,
@@ -598,26 +601,28 @@ def stream_add_rmsnorm(x, adds=(), normed=None, normed_weight=None, vec=None, we
 
 
 def latent_norm_append(p, offset: int, rank: int, weight, eps: float, cache, block_table, ctx_len, q_len, emit_rows: bool = False,
-                       rot_dim: int = 0, cos=None, sin=None, q_rank: int = 0, q_weight=None):
+                       rot_dim: int = 0, cos=None, sin=None, q_rank: int = 0, q_weight=None, interleaved: bool = False):
     """``emit_rows``: also return the cache rows in token order ``[B, T, 1, rank + rot_dim]`` (zeros past ``q_len``).  With ``q_rank``
     the result is ``(rows, normalised query latent [B, T, q_rank])``."""
     if _mix_cuda(p) and p.stride(-1) == 1 and cache.dtype == p.dtype and cache.is_contiguous() and rot_dim % 2 == 0:
         stats["latent_norm_append"] += 1
         f32 = lambda t: None if t is None else t.float().contiguous()          # noqa: E731
         rows, cq = _C().latent_norm_append(p, int(offset), int(rank), f32(weight), float(eps), cache, _i32(block_table),
-                                           _i32(ctx_len), _i32(q_len), bool(emit_rows), int(rot_dim), f32(cos), f32(sin), int(q_rank), f32(q_weight))
+                                           _i32(ctx_len), _i32(q_len), bool(emit_rows), int(rot_dim), f32(cos), f32(sin), int(q_rank), f32(q_weight),
+                                           bool(interleaved))
         return (rows, cq) if q_rank else rows
     return ref.latent_norm_append(p, offset, rank, weight, eps, cache, block_table, ctx_len, q_len, emit_rows, rot_dim, cos, sin, q_rank,
-                                  q_weight)
+                                  q_weight, interleaved)
 
 
-def rope_half_tail(src, dst, rot_dim: int, cos, sin):
-    """Rotate-half rotation of the last ``rot_dim`` channels of every head of ``src`` into the last ``rot_dim`` channels of ``dst``."""
+def rope_tail(src, dst, rot_dim: int, cos, sin, interleaved: bool = False):
+    """Rotation (rotate-half layout, or pairs (2i, 2i+1) with ``interleaved``) of the last ``rot_dim`` channels of every head of ``src`` into
+    the last ``rot_dim`` channels of ``dst``."""
     if _mix_cuda(src) and dst.dtype == src.dtype and src.is_contiguous() and dst.is_contiguous() and rot_dim % 2 == 0:
-        stats["rope_half_tail"] += 1
-        _C().rope_half_tail(src, dst, int(rot_dim), cos.float().contiguous(), sin.float().contiguous())
+        stats["rope_tail"] += 1
+        _C().rope_tail(src, dst, int(rot_dim), cos.float().contiguous(), sin.float().contiguous(), bool(interleaved))
         return dst
-    return ref.rope_half_tail(src, dst, rot_dim, cos, sin)
+    return ref.rope_tail(src, dst, rot_dim, cos, sin, interleaved)
 
 
 def stream_norm_conv(x, adds, weight, conv_w, state, slots, ctx_len, q_len, eps: float, lp_dtype=None):
@@ -780,6 +785,31 @@ def decay_scan(p, decay, state, slots, ctx_len, q_len, n_heads: int, D: int, Dv:
         stats["decay_scan"] += 1
         return _C().decay_scan(p, decay, state, _i32(slots), _i32(ctx_len), _i32(q_len), int(n_heads), int(D), int(Dv), bool(silu))
     return ref.decay_scan(p, decay, state, slots, ctx_len, q_len, n_heads, D, Dv, silu)
+
+
+def bigram_embed(ids, embed_w, bigram_w, scale: float, mul_prev: int, mul_cur: int, state, slots, ctx_len, q_len, lp_dtype=None):
+    """Scaled token embedding + bigram embedding as the fp32 stream and its low-precision copy, carried token advanced, ONE kernel
+    (definition: ops/reference.py)."""
+    if (_mix_cuda(embed_w) and embed_w.is_contiguous() and (bigram_w is None or (bigram_w.dtype == embed_w.dtype and bigram_w.is_contiguous()))
+            and ids.dim() == 2):
+        stats["bigram_embed"] += 1
+        lp = lp_dtype == torch.bfloat16
+        x, x_lp = _C().bigram_embed(_i32(ids), embed_w, bigram_w, float(scale), int(mul_prev), int(mul_cur), state, _i32(slots), _i32(ctx_len),
+                                    _i32(q_len), lp)
+        return x, x_lp
+    return ref.bigram_embed(ids, embed_w, bigram_w, scale, mul_prev, mul_cur, state, slots, ctx_len, q_len, lp_dtype)
+
+
+MLSTM_SLICE = ref.MLSTM_SLICE
+
+
+def mlstm_scan(p, gate_at: int, i_bias, f_bias, cap: float, state, key_sum, run_max, slots, ctx_len, q_len, n_heads: int, D: int, Dv: int):
+    """Matrix memory with exponential input gates, gates and denominator included, ONE kernel (definition: ops/reference.py)."""
+    if _mix_cuda(p) and p.stride(-1) == 1 and state.dtype == torch.float32 and D <= 256:
+        stats["mlstm_scan"] += 1
+        return _C().mlstm_scan(p, int(gate_at), i_bias, f_bias, float(cap), state, key_sum, run_max, _i32(slots), _i32(ctx_len), _i32(q_len),
+                               int(n_heads), int(D), int(Dv))
+    return ref.mlstm_scan(p, gate_at, i_bias, f_bias, cap, state, key_sum, run_max, slots, ctx_len, q_len, n_heads, D, Dv)
 
 
 def table_route(table, token_ids, q_len):

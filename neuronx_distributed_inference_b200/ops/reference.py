@@ -437,41 +437,47 @@ def short_conv_update(u, state, slots, ctx_len, q_len):
     state[slots.long()] = torch.where(keep, new, state[slots.long()])
 
 
-def rope_partial_interleaved(x, cos, sin):
-    """x [B, T, H, D]; cos/sin [B, T, R/2]: channel pairs (2i, 2i+1), i < R/2, are rotated, the rest pass through."""
-    R = 2 * cos.shape[-1]
-    xr = x[..., :R].float().reshape(*x.shape[:-1], R // 2, 2)
-    c, s = cos.float().unsqueeze(2), sin.float().unsqueeze(2)
+def rotate_pair_rows(x, cos, sin):
+    """x [..., R] with cos / sin broadcastable to [..., R / 2]: channel ``2i`` pairs with ``2i + 1``.  fp32."""
+    xr = x.float().reshape(*x.shape[:-1], x.shape[-1] // 2, 2)
     a, b = xr[..., 0], xr[..., 1]
-    rot = torch.stack([a * c - b * s, b * c + a * s], -1).reshape(*x.shape[:-1], R)
-    return torch.cat([rot, x[..., R:].float()], -1)
+    return torch.stack([a * cos - b * sin, b * cos + a * sin], -1).reshape(x.shape)
+
+
+def rope_partial(x, cos, sin, half: bool = False):
+    """x [B, T, H, D]; cos/sin [B, T, R/2]: the first R channels are rotated in pairs (2i, 2i+1), or (i, i + R/2) with ``half``; the rest
+    pass through."""
+    R = 2 * cos.shape[-1]
+    rows = rotate_half_rows if half else rotate_pair_rows
+    return torch.cat([rows(x[..., :R], cos.float().unsqueeze(2), sin.float().unsqueeze(2)), x[..., R:].float()], -1)
 
 
 def conv_qknorm_rope_append(qkv, conv_w, state, slots, ctx_len, q_len, q_norm_w, k_norm_w, eps: float, n_q: int, n_kv: int,
-                            D: int, Dv: int, cos, sin, k_cache, v_cache, block_table, out_dtype=None):
+                            D: int, Dv: int, cos, sin, k_cache, v_cache, block_table, out_dtype=None, half: bool = False):
     """Fused front half of a convolved-projection attention layer.  ``qkv`` [B, T, >= n_q*D + n_kv*(D+Dv)] holds the biased q | k | v
     projections (``n_kv = 0``: queries only, for a layer that reads another layer's cache; a norm weight of ``None`` skips that row
     norm, ``cos = None`` skips the rotation).  Steps: short causal convolution of every
     channel (carried inputs in ``state``), RMS norm of the WHOLE q row and of the WHOLE k row (plain weights), rotation of the first
     ``2 * cos.shape[-1]`` channels of every q / k head, and the write of k (normed, rotated) and v (convolved only) into the paged
-    caches ``[blocks, page, n_kv, D | Dv]`` at position ``ctx_len + t``.  Returns q [B, T, n_q, D]."""
+    caches ``[blocks, page, n_kv, D | Dv]`` at position ``ctx_len + t``.  Returns q [B, T, n_q, D].  ``conv_w = None``: no convolution
+    (no carried inputs either); ``half``: rotation pairs (i, i + R/2) instead of (2i, 2i+1)."""
     B, T = qkv.shape[:2]
     Cq, Ck, Cv = n_q * D, n_kv * D, n_kv * Dv
     C = Cq + Ck + Cv
-    y = short_conv(qkv[..., :C], conv_w, None, state, slots, ctx_len, q_len)
+    y = qkv[..., :C].float() if conv_w is None else short_conv(qkv[..., :C], conv_w, None, state, slots, ctx_len, q_len)
     q = y[..., :Cq]
     if q_norm_w is not None:
         q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps) * q_norm_w.float()
     q = q.view(B, T, n_q, D)
     if cos is not None:
-        q = rope_partial_interleaved(q, cos, sin)
+        q = rope_partial(q, cos, sin, half)
     if n_kv:
         k = y[..., Cq:Cq + Ck]
         if k_norm_w is not None:
             k = k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps) * k_norm_w.float()
         k = k.view(B, T, n_kv, D)
         if cos is not None:
-            k = rope_partial_interleaved(k, cos, sin)
+            k = rope_partial(k, cos, sin, half)
         v = y[..., Cq + Ck:].view(B, T, n_kv, Dv)
         page = k_cache.shape[1]
         t = torch.arange(T, device=qkv.device).view(1, T)
@@ -618,12 +624,13 @@ def rotate_half_rows(x, cos, sin):
 
 
 def latent_norm_append(p, offset: int, rank: int, weight, eps: float, cache, block_table, ctx_len, q_len, emit_rows: bool = False,
-                       rot_dim: int = 0, cos=None, sin=None, q_rank: int = 0, q_weight=None):
+                       rot_dim: int = 0, cos=None, sin=None, q_rank: int = 0, q_weight=None, interleaved: bool = False):
     """Channels ``[offset, offset + rank)`` of the projection rows ``p`` [B, T, C] are RMS-normalised (fp32, ``weight`` [rank]) and
     written to the paged latent cache ``[blocks, page, 1, rank + rot_dim]`` at positions ``ctx_len + t`` for ``t < q_len``.
 
     ``rot_dim`` > 0: the next ``rot_dim`` channels (not normalised) are one rotated key part shared by all heads; they are rotated in
-    the rotate-half layout with ``cos`` / ``sin`` [B, T, rot_dim / 2] and stored behind the latent in the same cache row.
+    the rotate-half layout (``interleaved``: pairs (2i, 2i+1)) with ``cos`` / ``sin`` [B, T, rot_dim / 2] and stored behind the latent
+    in the same cache row.
     ``q_rank`` > 0: channels ``[0, q_rank)`` are a query latent; its RMS norm times ``q_weight`` is returned as well
     (``(rows, q_latent [B, T, q_rank])`` instead of ``rows``)."""
     B, T = p.shape[:2]
@@ -631,7 +638,8 @@ def latent_norm_append(p, offset: int, rank: int, weight, eps: float, cache, blo
     c = p[..., offset:offset + rank].float()
     c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
     if rot_dim:
-        c = torch.cat([c, rotate_half_rows(p[..., offset + rank:offset + rank + rot_dim], cos.float(), sin.float())], -1)
+        rows_of = rotate_pair_rows if interleaved else rotate_half_rows
+        c = torch.cat([c, rows_of(p[..., offset + rank:offset + rank + rot_dim], cos.float(), sin.float())], -1)
     pos = ctx_len.long().view(B, 1) + torch.arange(T, device=p.device).view(1, T)
     live = torch.arange(T, device=p.device).view(1, T) < q_len.long().view(B, 1)
     width = block_table.shape[1]
@@ -646,11 +654,13 @@ def latent_norm_append(p, offset: int, rank: int, weight, eps: float, cache, blo
     return rows
 
 
-def rope_half_tail(src, dst, rot_dim: int, cos, sin):
-    """The last ``rot_dim`` channels of every head of ``src`` [B, T, H, Ds] are rotated (rotate-half layout, ``cos`` / ``sin``
-    [B, T, rot_dim / 2], fp32) and written to the last ``rot_dim`` channels of the heads of ``dst`` [B, T, H, Dd]."""
-    dst[..., dst.shape[-1] - rot_dim:] = rotate_half_rows(src[..., src.shape[-1] - rot_dim:], cos.float().unsqueeze(2),
-                                                          sin.float().unsqueeze(2)).to(dst.dtype)
+def rope_tail(src, dst, rot_dim: int, cos, sin, interleaved: bool = False):
+    """The last ``rot_dim`` channels of every head of ``src`` [B, T, H, Ds] are rotated (rotate-half layout, or pairs (2i, 2i+1) with
+    ``interleaved``; ``cos`` / ``sin`` [B, T, rot_dim / 2], fp32) and written to the last ``rot_dim`` channels of the heads of ``dst``
+    [B, T, H, Dd]."""
+    rows_of = rotate_pair_rows if interleaved else rotate_half_rows
+    dst[..., dst.shape[-1] - rot_dim:] = rows_of(src[..., src.shape[-1] - rot_dim:], cos.float().unsqueeze(2),
+                                                 sin.float().unsqueeze(2)).to(dst.dtype)
     return dst
 
 
@@ -805,9 +815,10 @@ def gated_delta_scan(qkv, beta_raw, a_raw, A_log, dt_bias, state, slots, ctx_len
 
 def head_rmsnorm_gate(y, weight, heads: int, eps: float, gate, act: str = "silu", out_dtype=None):
     """``y`` [..., heads * Dv] fp32: every head is divided by its root mean square over ``Dv``, times ``weight`` [Dv] (shared by the
-    heads), times ``act(gate)`` (``gate`` [..., heads * Dv], possibly a strided slice of a wider row); the gate comes AFTER the norm."""
+    heads) or [heads * Dv], times ``act(gate)`` (``gate`` [..., heads * Dv], possibly a strided slice of a wider row); the gate comes
+    AFTER the norm."""
     Dv = y.shape[-1] // heads
-    yf = _norm_rows(y.float().reshape(*y.shape[:-1], heads, Dv), False, eps) * weight.float()
+    yf = _norm_rows(y.float().reshape(*y.shape[:-1], heads, Dv), False, eps) * weight.float().reshape(-1, Dv)
     return (yf.reshape(y.shape) * activation(gate.float(), act)).to(out_dtype or y.dtype)
 
 
@@ -920,6 +931,77 @@ def decay_scan(p, decay, state, slots, ctx_len, q_len, n_heads: int, D: int, Dv:
         S = torch.where((t < q_len).view(B, 1, 1, 1), S * lam + v[:, t, :, :, None] * k[:, t, :, None, :], S)
         out.append((S * q[:, t, :, None, :]).sum(-1))
     state[slots.long()] = torch.where((q_len > 0).view(B, 1, 1, 1), S, state[slots.long()].float()).to(state.dtype)
+    return torch.stack(out, 1).reshape(B, T, H * Dv)
+
+
+# ---- embeddings with a carried token, matrix memory with exponential gates ---------------------------------------------------------------
+def bigram_rows(ids, prev, ctx_len, buckets: int, mul_prev: int, mul_cur: int):
+    """Row of a bigram table for every token of ``ids`` [B, T]: ``(previous * mul_prev + current * mul_cur) mod buckets``; the first token
+    of a sequence has row ``buckets``.  ``prev`` [B]: the token before a portion (read when ``ctx_len > 0``)."""
+    ids = ids.long()
+    before = torch.cat([prev.long().view(-1, 1), ids[:, :-1]], 1)
+    rows = (before * int(mul_prev) + ids * int(mul_cur)) % int(buckets)
+    first = (ctx_len == 0).view(-1, 1) & (torch.arange(ids.shape[1], device=ids.device) == 0)
+    return torch.where(first, torch.full_like(rows, int(buckets)), rows)
+
+
+def bigram_embed(ids, embed_w, bigram_w, scale: float, mul_prev: int, mul_cur: int, state, slots, ctx_len, q_len, lp_dtype=None):
+    """``x = embed[id] * scale + bigram[row]`` in fp32 (``bigram_w`` [buckets + 1, W] or None: no such term; rows: :func:`bigram_rows`).
+    ``state`` [lines, 1] int32 carries the last token of every sequence and is advanced.  Rows past ``q_len`` are zero.
+    Returns ``(x, x cast to lp_dtype or None)``."""
+    B, T = ids.shape
+    live = torch.arange(T, device=ids.device).view(1, T) < q_len.long().view(B, 1)
+    x = embed_w[ids.long()].float() * scale
+    if bigram_w is not None:
+        line = slots.long()
+        x = x + bigram_w[bigram_rows(ids, state[line, 0], ctx_len, bigram_w.shape[0] - 1, mul_prev, mul_cur)].float()
+        last = ids.gather(1, (q_len.long() - 1).clamp_min(0).view(B, 1)).view(B).to(state.dtype)
+        state[line, 0] = torch.where(q_len > 0, last, state[line, 0])
+    x = torch.where(live.unsqueeze(-1), x, torch.zeros_like(x))
+    return x, (None if lp_dtype in (None, torch.float32) else x.to(lp_dtype))
+
+
+MLSTM_SLICE = 16         # value channels that share one copy of the key sum and of the running maximum (csrc/linear_scan.cu)
+
+
+def mlstm_scan(p, gate_at: int, i_bias, f_bias, cap: float, state, key_sum, run_max, slots, ctx_len, q_len, n_heads: int, D: int, Dv: int):
+    """Matrix memory with exponential input gates.  ``p`` [B, T, C] holds q | k | v at channel 0 and the raw input and forget gates (one
+    per head each) at channel ``gate_at``.  Per head, fp32::
+
+        i = cap tanh((raw_i + i_bias) / cap);   f = logsigmoid(cap tanh((raw_f + f_bias) / cap))
+        m' = max(f + m, i);   S' = exp(f + m - m') S + exp(i - m') v k^T;   n' = exp(f + m - m') n + exp(i - m') k
+        o = S' q / (max(|n' . q|, exp(-m')) + 1e-6)       with q scaled by D^-1/2
+
+    S, n and m start at zero.  ``state`` [lines, heads, Dv, D] holds S; ``key_sum`` [lines, heads, slices, D] and ``run_max`` [lines, heads,
+    slices] hold one copy of n and m for every ``MLSTM_SLICE`` value channels.  Returns o fp32 [B, T, heads * Dv]; padding steps leave the
+    state untouched."""
+    B, T = p.shape[:2]
+    H = n_heads
+    q, k, v = (t.reshape(B, T, H, -1).float() for t in p[..., :H * (2 * D + Dv)].split([H * D, H * D, H * Dv], -1))
+    q = q * D ** -0.5
+    raw = p[..., gate_at:gate_at + 2 * H].float()
+    gi = cap * torch.tanh((raw[..., :H] + i_bias.float()) / cap)
+    gf = F.logsigmoid(cap * torch.tanh((raw[..., H:] + f_bias.float()) / cap))
+    line = slots.long()
+    fresh = (ctx_len == 0).view(B, 1)
+    S = state[line].masked_fill(fresh.view(B, 1, 1, 1), 0.0)
+    n = key_sum[line][:, :, 0].masked_fill(fresh.view(B, 1, 1), 0.0)
+    m = run_max[line][:, :, 0].masked_fill(fresh, 0.0)
+    out = []
+    for t in range(T):
+        on = (t < q_len).view(B, 1)
+        new = torch.maximum(gf[:, t] + m, gi[:, t])
+        fade, put = torch.exp(gf[:, t] + m - new), torch.exp(gi[:, t] - new)
+        fade, put = torch.where(on, fade, torch.ones_like(fade)), torch.where(on, put, torch.zeros_like(put))
+        m = torch.where(on, new, m)
+        S = S * fade[..., None, None] + put[..., None, None] * v[:, t, :, :, None] * k[:, t, :, None, :]
+        n = n * fade[..., None] + put[..., None] * k[:, t]
+        den = torch.maximum((n * q[:, t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+        out.append((S * q[:, t, :, None, :]).sum(-1) / den.unsqueeze(-1))
+    live = (q_len > 0).view(B, 1)
+    state[line] = torch.where(live[..., None, None], S, state[line])
+    key_sum[line] = torch.where(live[..., None, None], n.unsqueeze(2).expand(-1, -1, key_sum.shape[2], -1), key_sum[line])
+    run_max[line] = torch.where(live[..., None], m.unsqueeze(2).expand(-1, -1, run_max.shape[2]), run_max[line])
     return torch.stack(out, 1).reshape(B, T, H * Dv)
 
 

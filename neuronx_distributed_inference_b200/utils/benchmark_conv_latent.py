@@ -147,7 +147,7 @@ def kernel_table(size, batch, prompt, hbm_gbs, tflops):
         c0 = rnd(B * nblk, page, 1, R)
         run(f"{phase}: like: latent_norm_append (latent norm only)", lambda: ops.latent_norm_append(p, Q, R, lw, 1e-5, c0, table, ctx, ql), N * R * 2 * 2)
         qf, a = rnd(B, T, H, D + rot), rnd(B, T, H, R + rot) * 0.2
-        run(f"{phase}: rope_half_tail (rotated query channels behind the absorbed ones)", lambda: ops.rope_half_tail(qf, a, rot, cos, sin), N * H * rot * 2 * 2)
+        run(f"{phase}: rope_tail (rotated query channels behind the absorbed ones)", lambda: ops.rope_tail(qf, a, rot, cos, sin), N * H * rot * 2 * 2)
         win = min(s["window"], keys)
         lat_flops = 2.0 * B * H * (2 * R + rot) * sum(min(t + 1 + ctx0, s["window"]) for t in range(T))
         run(f"{phase}: paged_window_attention (latent rows + rotated tail as keys, prefix as values, window {s['window']})",

@@ -103,7 +103,9 @@ MODEL_TYPES["sodudra"] = {"causal-lm": f"{_P}.sodudra.modeling_sodudra:NeuronSod
 MODEL_TYPES["tusipel"] = {"causal-lm": f"{_P}.tusipel.modeling_tusipel:NeuronTusipelForCausalLM"}
 MODEL_TYPES["zanivik"] = {"causal-lm": f"{_P}.zanivik.modeling_zanivik:NeuronZanivikForCausalLM"}
 MODEL_TYPES["balivik"] = {"causal-lm": f"{_P}.balivik.modeling_balivik:NeuronBalivikForCausalLM"}
-ARCHITECTURES = {"Fetodra": "fetodra", "Sodudra": "sodudra", "Tusipel": "tusipel", "Zanivik": "zanivik", "Balivik": "balivik"}
+MODEL_TYPES["navulorn"] = {"causal-lm": f"{_P}.navulorn.modeling_navulorn:NeuronNavulornForCausalLM"}
+ARCHITECTURES = {"Fetodra": "fetodra", "Sodudra": "sodudra", "Tusipel": "tusipel", "Zanivik": "zanivik", "Balivik": "balivik",
+                 "Navulorn": "navulorn"}
 TASK_TYPES = ("causal-lm", "image-text-to-text", "speech-to-text", "text-to-image", "audio-frame-classification", "audio-text-to-text")
 
 

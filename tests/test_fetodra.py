@@ -230,7 +230,7 @@ def test_rotation_pairs_and_partial_width():
     x, pos = torch.randn(5, 2, 8, dtype=torch.float64), torch.tensor([0, 1, 7, 300, 4000])
     want = oracle.rotate_interleaved(x, pos, 4, 100.0)
     ang = pos.double()[:, None] * (100.0 ** (-torch.arange(0, 4, 2).double() / 4))
-    got = ref.rope_partial_interleaved(x.unsqueeze(0), torch.cos(ang).unsqueeze(0), torch.sin(ang).unsqueeze(0))[0]
+    got = ref.rope_partial(x.unsqueeze(0), torch.cos(ang).unsqueeze(0), torch.sin(ang).unsqueeze(0))[0]
     assert torch.allclose(got, want.float(), atol=1e-6) and torch.equal(got[..., 4:], x[..., 4:].float())
 
 

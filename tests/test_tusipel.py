@@ -425,7 +425,7 @@ def test_scaled_rotation_tables_and_rotate_half_layout():
     c, s = oracle.yarn_tables(1005, rot)
     g = torch.Generator().manual_seed(2)
     src, dst = torch.randn(2, 5, 3, 12, generator=g), torch.zeros(2, 5, 3, 20)
-    ops.rope_half_tail(src, dst, 8, cos, sin)
+    ops.rope_tail(src, dst, 8, cos, sin)
     want = oracle.rotate_half(src[1, :, :, 4:].double(), c[1000:], s[1000:])
     assert torch.allclose(dst[1, :, :, 12:].double(), want, atol=1e-5) and torch.all(dst[..., :12] == 0)
 
@@ -530,7 +530,7 @@ def test_gpu_stack_schedules_mixed_batches_and_generation(tmp_path, dtype):
     eng, cfg, w = check_schedules(tmp_path, "cuda", dtype)
     check_mixed_batches(eng, cfg, w, dtype)
     check_generate(eng, cfg, w, dtype)
-    for k in ("stream_norm_conv", "short_conv_update", "latent_norm_append", "rope_half_tail", "conv_qknorm_rope_append", "paged_window_attention",
+    for k in ("stream_norm_conv", "short_conv_update", "latent_norm_append", "rope_tail", "conv_qknorm_rope_append", "paged_window_attention",
               "gated_act_mul", "clamped_glu", "router_topk", "identity_expert_add", "stream_add_rmsnorm"):
         assert ops.stats[k] > 0, k
     assert ops.stats["moe_plain_gated"] > 0                                # experts of sizes no tensor-core tile fits
@@ -606,8 +606,8 @@ def test_gpu_kernels_match_definitions():
         assert torch.allclose(c1.float(), c2.float().cpu(), atol=tol, rtol=1e-4) and torch.allclose(q1.float() * live, q2.float().cpu() * live, atol=tol * 2)
         src = rn(B, T, H, 12 + rot).to(dt)
         d1, d2 = torch.zeros(B, T, H, R + rot, dtype=dt), torch.zeros(B, T, H, R + rot, dtype=dt, device=dev)
-        ref.rope_half_tail(src, d1, rot, cos, sin)
-        ops.rope_half_tail(src.to(dev), d2, rot, *on(cos, sin))
+        ref.rope_tail(src, d1, rot, cos, sin)
+        ops.rope_tail(src.to(dev), d2, rot, *on(cos, sin))
         assert torch.allclose(d1.float(), d2.float().cpu(), atol=tol)
         # attention over those rows: window, values as the prefix of the key rows
         q = rn(B, T, H, R + rot).to(dt) * 0.3
