@@ -1103,14 +1103,14 @@ __global__ void __launch_bounds__(256) latent_norm_append_kernel(const T* __rest
 
 // dst[tok, h, Dd - rot + .] = rotate(src[tok, h, Ds - rot + .]); one thread per (token, head, pair)
 template <typename T>
-__global__ void __launch_bounds__(256) rope_tail_kernel(const T* __restrict__ src, T* __restrict__ dst, const float* __restrict__ cosv,
+__global__ void __launch_bounds__(256) rope_tail_kernel(const T* __restrict__ src, long long src_st, T* __restrict__ dst, const float* __restrict__ cosv,
                                                              const float* __restrict__ sinv, long long n, int H, int Ds, int Dd, int rot,
                                                              int interleaved) {
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= n) return;
   const int half = rot / 2, i = (int)(idx % half);
   const long long th = idx / half, tok = th / H;
-  const T* sr = src + th * Ds + (Ds - rot);
+  const T* sr = src + tok * src_st + (th % H) * Ds + (Ds - rot);
   T* dr = dst + th * Dd + (Dd - rot);
   const int c0 = interleaved ? 2 * i : i, c1 = interleaved ? 2 * i + 1 : half + i;
   const float u = ldf(sr + c0), v = ldf(sr + c1);
@@ -2229,13 +2229,13 @@ void latent_norm_append_launch(const void* p, long long p_sb, long long p_st, co
                                                            (float*)q_out, (int)interleaved);
 }
 
-void rope_tail_launch(const void* src, void* dst, const float* cos, const float* sin, long long tokens, int H, int Ds, int Dd, int rot,
+void rope_tail_launch(const void* src, long long src_st, void* dst, const float* cos, const float* sin, long long tokens, int H, int Ds, int Dd, int rot,
                       bool interleaved, bool lp, cudaStream_t st) {
   const long long n = tokens * H * (rot / 2);
   if (n <= 0) return;
   const unsigned grid = (unsigned)((n + 255) / 256);
-  if (lp) rope_tail_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>((const __nv_bfloat16*)src, (__nv_bfloat16*)dst, cos, sin, n, H, Ds, Dd, rot, (int)interleaved);
-  else rope_tail_kernel<float><<<grid, 256, 0, st>>>((const float*)src, (float*)dst, cos, sin, n, H, Ds, Dd, rot, (int)interleaved);
+  if (lp) rope_tail_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>((const __nv_bfloat16*)src, src_st, (__nv_bfloat16*)dst, cos, sin, n, H, Ds, Dd, rot, (int)interleaved);
+  else rope_tail_kernel<float><<<grid, 256, 0, st>>>((const float*)src, src_st, (float*)dst, cos, sin, n, H, Ds, Dd, rot, (int)interleaved);
 }
 
 void stream_norm_conv_launch(const StreamConvParams& p, bool out_lp, cudaStream_t st) {

@@ -37,8 +37,9 @@ void latent_norm_append_launch(const void* p, long long p_sb, long long p_st, co
                                void* rows_out, int rot, const float* cos, const float* sin, const void* q_in, int q_rank, const float* q_w,
                                void* q_out, bool interleaved, cudaStream_t st);      // rows_out: [B, T, R + rot] copy of the live rows in token order, or null
 
-// dst[b, t, h, Dd - rot ...] = rotate(src[b, t, h, Ds - rot ...]) with cos / sin [B * T, rot / 2]; pairs as in latent_norm_append
-void rope_tail_launch(const void* src, void* dst, const float* cos, const float* sin, long long tokens, int H, int Ds, int Dd, int rot,
+// dst[b, t, h, Dd - rot ...] = rotate(src[b, t, h, Ds - rot ...]) with cos / sin [B * T, rot / 2]; pairs as in latent_norm_append;
+// src_st: elements between tokens of src (heads dense)
+void rope_tail_launch(const void* src, long long src_st, void* dst, const float* cos, const float* sin, long long tokens, int H, int Ds, int Dd, int rot,
                       bool interleaved, bool lp, cudaStream_t st);
 
 // s = x + [y1] + [y2]; h = rms_unit(s) * w; out = h + sum_j cw[:, j] * h_(t - K + 1 + j), the rows before a portion from the fp32 state

@@ -618,7 +618,8 @@ def latent_norm_append(p, offset: int, rank: int, weight, eps: float, cache, blo
 def rope_tail(src, dst, rot_dim: int, cos, sin, interleaved: bool = False):
     """Rotation (rotate-half layout, or pairs (2i, 2i+1) with ``interleaved``) of the last ``rot_dim`` channels of every head of ``src`` into
     the last ``rot_dim`` channels of ``dst``."""
-    if _mix_cuda(src) and dst.dtype == src.dtype and src.is_contiguous() and dst.is_contiguous() and rot_dim % 2 == 0:
+    rows = src.stride(3) == 1 and src.stride(2) == src.shape[3] and (src.shape[0] == 1 or src.stride(0) == src.shape[1] * src.stride(1))
+    if _mix_cuda(src) and dst.dtype == src.dtype and rows and dst.is_contiguous() and rot_dim % 2 == 0:
         stats["rope_tail"] += 1
         _C().rope_tail(src, dst, int(rot_dim), cos.float().contiguous(), sin.float().contiguous(), bool(interleaved))
         return dst
