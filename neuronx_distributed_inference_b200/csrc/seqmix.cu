@@ -250,6 +250,107 @@ __global__ void __launch_bounds__(256) conv_qknorm_rope_append_pair_kernel(ConvQ
   for (int c = 2 * threadIdx.x; c < Cv; c += 2 * blockDim.x) st2(vo + c, buf[Cq + Ck + c], buf[Cq + Ck + c + 1]);
 }
 
+// No convolution, head and rotation sizes in multiples of 8: eight channels per access, both row sums in one reduction; the raw row waits in
+// shared memory for its norm and its rotation partners.
+__device__ __forceinline__ void ld8(const float* p, float* v) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void ld8(const __nv_bfloat16* p, float* v) {
+  const uint4 r = *reinterpret_cast<const uint4*>(p);
+  v[0] = bf16lo(r.x); v[1] = bf16hi(r.x); v[2] = bf16lo(r.y); v[3] = bf16hi(r.y);
+  v[4] = bf16lo(r.z); v[5] = bf16hi(r.z); v[6] = bf16lo(r.w); v[7] = bf16hi(r.w);
+}
+__device__ __forceinline__ void st8(float* p, const float* v) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void st8(__nv_bfloat16* p, const float* v) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) qknorm_rope_append_vec_kernel(ConvQkParams p) {
+  extern __shared__ __align__(16) float buf[];      // [Cq + Ck] raw row
+  __shared__ float red[16];
+  const int b = blockIdx.y, t = blockIdx.x;
+  const int Cq = p.n_q * p.D, Ck = p.n_kv * p.D, Cv = p.n_kv * p.Dv;
+  const long long tok = (long long)b * p.T + t;
+  T* qo = (T*)p.q_out + tok * Cq;
+  if (t >= p.q_len[b]) return;
+  const T* u = (const T*)p.p + (long long)b * p.p_sb + (long long)t * p.p_st;
+  const int pos = p.ctx_len[b] + t;
+  long long slot = 0;
+  if (p.n_kv) slot = (long long)p.block_table[(long long)b * p.max_blocks + pos / p.page] * p.page + pos % p.page;
+  T* ko = (T*)p.k_cache + slot * Ck;
+  T* vo = (T*)p.v_cache + slot * Cv;
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * 8; c < Cq + Ck; c += 256 * 8) {
+    float v[8];
+    ld8(u + c, v);
+    st8(buf + c, v);
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += v[e] * v[e];
+    if (c < Cq) sq += ss; else sk += ss;
+  }
+  for (int c = threadIdx.x * 8; c < Cv; c += 256 * 8) {
+    float v[8];
+    ld8(u + Cq + Ck + c, v);
+    st8(vo + c, v);
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) { red[threadIdx.x >> 5] = sq; red[8 + (threadIdx.x >> 5)] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) { sq += red[w]; sk += red[8 + w]; }
+  const float rq = p.q_norm_w ? 1.f / sqrtf(sq / (float)Cq + p.eps) : 1.f;
+  const float rk = (Ck && p.k_norm_w) ? 1.f / sqrtf(sk / (float)Ck + p.eps) : 1.f;
+  const int hr = p.R / 2;
+  const float* cs = p.cos + tok * hr;
+  const float* sn = p.sin + tok * hr;
+  for (int c = threadIdx.x * 8; c < Cq + Ck; c += 256 * 8) {
+    const bool isq = c < Cq;
+    const int cc = isq ? c : c - Cq, d = cc % p.D;
+    const float r = isq ? rq : rk;
+    const float* nw = isq ? p.q_norm_w : p.k_norm_w;
+    float v[8], g[8];
+    ld8(buf + c, v);
+    if (nw) {
+      ld8(nw + cc, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] *= r * g[e];
+    }
+    if (d < p.R) {
+      if (p.half) {
+        const bool second = d >= hr;
+        const int step = second ? -hr : hr, i = second ? d - hr : d;
+        float o[8], co[8], si[8];
+        ld8(buf + c + step, o);
+        if (nw) {
+          ld8(nw + cc + step, g);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) o[e] *= r * g[e];
+        }
+        ld8(cs + i, co);
+        ld8(sn + i, si);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = second ? v[e] * co[e] + o[e] * si[e] : v[e] * co[e] - o[e] * si[e];
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; e += 2) {
+          const float co = cs[(d + e) >> 1], si = sn[(d + e) >> 1], a = v[e], bb = v[e + 1];
+          v[e] = a * co - bb * si;
+          v[e + 1] = bb * co + a * si;
+        }
+      }
+    }
+    st8((isq ? qo : ko) + cc, v);
+  }
+}
+
 // ---- soft-capped kept-prefix sliding-window attention over the paged cache ---------------------------------------------------
 template <typename T> struct Vec;                     // 16-byte vectors of the activation type
 template <> struct Vec<float> { static constexpr int N = 4; };
@@ -277,14 +378,14 @@ __device__ __forceinline__ float dot_row(const float* qs, const T* k, int D, boo
 }
 
 constexpr int ATT_WARPS = 4;
-constexpr int ATT_VPL = SEQMIX_MAX_VDIM / 32;      // value channels per lane
 
 // SPLIT = false: warp w of a block owns query blockIdx.x * 4 + w.  SPLIT = true: the warps share query blockIdx.x, warp w takes
 // key chunks w, w + 4, ... and the partial (max, sum, acc) are merged through shared memory (few queries, long ranges: decode).
 // MAPS = 2 (differential attention): a head has two queries and two keys per token over the same values; a query's warp attends with one
 // after the other (SPLIT: half of the warps with each), and the epilogue subtracts, normalises and scales.
-template <typename T, bool SPLIT, int MAPS>
-__global__ void __launch_bounds__(SPLIT ? 1024 : ATT_WARPS * 32) paged_window_attention_kernel(WindowAttnParams p) {
+// ATT_VPL: value channels per lane.
+template <typename T, bool SPLIT, int MAPS, int ATT_VPL>
+__global__ void __launch_bounds__(SPLIT ? (ATT_VPL > 8 ? 512 : 1024) : ATT_WARPS * 32) paged_window_attention_kernel(WindowAttnParams p) {
   extern __shared__ float smem[];      // [warps][D] scaled queries, then [warps][Dv + 2] partials
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
   const long long nq = (long long)p.B * p.T * p.Hq;
@@ -2360,6 +2461,17 @@ void conv_qknorm_rope_append_launch(const ConvQkParams& p, bool lp, cudaStream_t
   const size_t smem = sizeof(float) * (size_t)(p.n_q * p.D + p.n_kv * (p.D + p.Dv));
   dim3 grid(p.T, p.B);
   const size_t esz = lp ? 2 : 4;
+  auto al16 = [](const void* q) { return ((uintptr_t)q & 15) == 0; };
+  if (!p.conv_w && p.D % 8 == 0 && p.Dv % 8 == 0 && p.R % (p.half ? 16 : 8) == 0 && (p.p_sb * esz) % 16 == 0 && (p.p_st * esz) % 16 == 0 && al16(p.p) &&
+      al16(p.q_out) && al16(p.k_cache) && al16(p.v_cache) && al16(p.q_norm_w) && al16(p.k_norm_w) && al16(p.cos) && al16(p.sin)) {
+    const size_t rows = sizeof(float) * (size_t)(p.n_q + p.n_kv) * p.D;
+    auto run = [&](auto kernel) {
+      opt_in_smem(kernel, rows);
+      kernel<<<grid, 256, rows, st>>>(p);
+    };
+    if (lp) run(qknorm_rope_append_vec_kernel<__nv_bfloat16>); else run(qknorm_rope_append_vec_kernel<float>);
+    return;
+  }
   const bool pairs = p.Dv % 2 == 0 && p.R % 2 == 0 && p.p_sb % 2 == 0 && p.p_st % 2 == 0 && ((uintptr_t)p.p % (2 * esz)) == 0;
   auto go = [&](auto kernel) {
     opt_in_smem(kernel, smem);
@@ -2419,7 +2531,8 @@ void paged_window_attention_launch(const WindowAttnParams& p, bool lp, cudaStrea
   if (p.window > 0) span = std::min<long long>(span, (long long)p.window + p.keep_first);
   if (p.chunk > 0) span = std::min<long long>(span, (long long)p.chunk);
   const int maps = two ? 2 : 1;          // two maps: half of the warps each
-  const int nwarps = split ? maps * (int)std::min<long long>(32 / maps, std::max<long long>(ATT_WARPS, (span + 31) / 32)) : ATT_WARPS;
+  const bool wide = p.Dv > SEQMIX_MAX_VDIM;
+  const int nwarps = split ? maps * (int)std::min<long long>((wide ? 16 : 32) / maps, std::max<long long>(ATT_WARPS, (span + 31) / 32)) : ATT_WARPS;
   const size_t smem = sizeof(float) * (size_t)(nwarps * (p.D + p.Dv + 2));
   const unsigned grid = (unsigned)(split ? nq : (nq + ATT_WARPS - 1) / ATT_WARPS);
   auto go = [&](auto kernel) {
@@ -2429,9 +2542,11 @@ void paged_window_attention_launch(const WindowAttnParams& p, bool lp, cudaStrea
   auto pick = [&](auto tag) {
     using T = decltype(tag);
     if (two) {
-      if (split) go(paged_window_attention_kernel<T, true, 2>); else go(paged_window_attention_kernel<T, false, 2>);
+      if (split) go(paged_window_attention_kernel<T, true, 2, 8>); else go(paged_window_attention_kernel<T, false, 2, 8>);
+    } else if (wide) {
+      if (split) go(paged_window_attention_kernel<T, true, 1, 16>); else go(paged_window_attention_kernel<T, false, 1, 16>);
     } else {
-      if (split) go(paged_window_attention_kernel<T, true, 1>); else go(paged_window_attention_kernel<T, false, 1>);
+      if (split) go(paged_window_attention_kernel<T, true, 1, 8>); else go(paged_window_attention_kernel<T, false, 1, 8>);
     }
   };
   if (lp) pick(__nv_bfloat16{}); else pick(float{});

@@ -8,7 +8,8 @@
 namespace nxdi {
 
 constexpr int SEQMIX_MAX_TAPS = 8;       // short convolutions: taps per channel
-constexpr int SEQMIX_MAX_VDIM = 256;     // attention: value channels per head
+constexpr int SEQMIX_MAX_VDIM = 256;     // differential attention, per-head norms: value channels per head
+constexpr int SEQMIX_MAX_ATT_VDIM = 512; // window attention: value channels per head (latent rows)
 constexpr int SEQMIX_MAX_STATE = 256;    // scan: state size per head
 constexpr int SEQMIX_MAX_STREAMS = 8;    // residual streams per token
 

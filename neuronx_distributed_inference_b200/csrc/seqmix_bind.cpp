@@ -166,7 +166,7 @@ at::Tensor paged_window_attention(const at::Tensor& q, const at::Tensor& k_cache
   // value_dim: the value of a key is the first value_dim channels of its row in v_cache
   const int64_t G = k_cache.size(2), Dv = value_dim;
   TORCH_CHECK(Dv >= 1 && Dv <= v_cache.size(3) && chunk >= 0 && !(chunk > 0 && window > 0), "paged_window_attention: value size / mask");
-  TORCH_CHECK(Hq % G == 0 && Dv <= SEQMIX_MAX_VDIM, "paged_window_attention: heads must divide, value size <= ", SEQMIX_MAX_VDIM);
+  TORCH_CHECK(Hq % G == 0 && Dv <= SEQMIX_MAX_ATT_VDIM, "paged_window_attention: heads must divide, value size <= ", SEQMIX_MAX_ATT_VDIM);
   TORCH_CHECK(block_table.is_cuda() && block_table.scalar_type() == at::kInt && block_table.is_contiguous() && block_table.dim() == 2 &&
               block_table.size(0) == B);
   check_i32(ctx, B, "ctx_len");
@@ -696,7 +696,7 @@ std::tuple<at::Tensor, at::Tensor, at::Tensor> router_topk(const at::Tensor& x, 
 void rope_tail(const at::Tensor& src, at::Tensor dst, int64_t rot, const at::Tensor& cos, const at::Tensor& sin, bool interleaved) {
   check_act(src, "rope_tail source");
   TORCH_CHECK(src.dim() == 4 && dst.dim() == 4 && src.stride(3) == 1 && src.stride(2) == src.size(3) &&
-              (src.size(0) == 1 || src.stride(0) == src.size(1) * src.stride(1)) && dst.is_contiguous() && dst.is_cuda() && dst.scalar_type() == src.scalar_type() &&
+              (src.size(0) == 1 || src.size(1) == 1 || src.stride(0) == src.size(1) * src.stride(1)) && dst.is_contiguous() && dst.is_cuda() && dst.scalar_type() == src.scalar_type() &&
               src.size(0) == dst.size(0) && src.size(1) == dst.size(1) && src.size(2) == dst.size(2) && rot % 2 == 0 && rot <= src.size(3) &&
               rot <= dst.size(3), "rope_tail: [B, T, H, D] tensors of one type");
   check_f32(cos, "cos");
@@ -704,7 +704,7 @@ void rope_tail(const at::Tensor& src, at::Tensor dst, int64_t rot, const at::Ten
   const int64_t tokens = src.size(0) * src.size(1);
   TORCH_CHECK(cos.numel() == tokens * (rot / 2) && sin.numel() == cos.numel(), "cos / sin [B, T, rot / 2]");
   c10::cuda::CUDAGuard guard(src.device());
-  rope_tail_launch(src.data_ptr(), src.stride(1), dst.data_ptr(), cos.data_ptr<float>(), sin.data_ptr<float>(), tokens, (int)src.size(2), (int)src.size(3),
+  rope_tail_launch(src.data_ptr(), src.size(1) == 1 ? src.stride(0) : src.stride(1), dst.data_ptr(), cos.data_ptr<float>(), sin.data_ptr<float>(), tokens, (int)src.size(2), (int)src.size(3),
                    (int)dst.size(3), (int)rot, interleaved, is_lp(src), stream());
 }
 

@@ -31,6 +31,7 @@ from ... import ops
 from ...config import InferenceConfig, NeuronConfig
 from ...modules.attention.conv_window_attention import ConvWindowAttention
 from ...modules.attention.latent_attention import LatentSinkAttention
+from ...modules.checkpoint import stack_rows
 from ...modules.kvcache import LayeredBlockKVCacheManager
 from ...modules.mlp import GatedMLP
 from ...modules.moe import ExpertMLPs, MoE, RouterTopK
@@ -201,7 +202,7 @@ class NeuronNavulornForCausalLM(NeuronBaseForCausalLM):
             x, y, m = a + "mix.", b + "mixer.", spec["mixer"]
             parts = lambda *names: [sd[x + n] for n in names]          # noqa: E731
             if spec["type"] == "attention":
-                out[y + "in_proj.weight"] = torch.cat(parts("q", "k", "v", "g"), 0)
+                out[y + "in_proj.weight"] = stack_rows(*parts("q", "k", "v", "g"))
                 out[y + "q_norm_weight"], out[y + "k_norm_weight"] = sd[x + "q.norm"], sd[x + "k.norm"]
                 out[y + "o_proj.weight"] = sd[x + "o"]
             elif spec["type"] == "latent_attention":
@@ -212,7 +213,7 @@ class NeuronNavulornForCausalLM(NeuronBaseForCausalLM):
                 out[y + "v_up"] = sd[x + "uv"].reshape(H, -1, R)
                 out[y + "o_proj.weight"] = sd[x + "o"]
             else:
-                out[y + "in_proj.weight"] = RaggedMatrixMemoryMixer.stack(*parts("q", "k", "v", "g", "i", "f"))
+                out[y + "in_proj.weight"] = stack_rows(*parts("q", "k", "v", "g", "i", "f"))
                 out[y + "i_bias"], out[y + "f_bias"] = sd[x + "i.b"], sd[x + "f.b"]
                 out[y + "norm_weight"], out[y + "out_proj.weight"] = sd[x + "norm"], sd[x + "o"]
             f = spec.get("mlp")

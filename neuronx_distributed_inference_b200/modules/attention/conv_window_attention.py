@@ -81,7 +81,10 @@ class ConvWindowAttention(nn.Module):
         self.Ckv = num_kv_heads * (head_dim + v_head_dim) if self.owns_kv else 0
         self.Co = num_heads * v_head_dim
         self.Cg = num_heads if self.head_gate else self.Co if out_gate else 0
-        self.in_proj = ColumnParallelLinear(hidden_size, self.Cq + self.Ckv + self.Cg, bias=bias, gather_output=False, dtype=dtype,
+        in_width = self.Cq + self.Ckv + self.Cg
+        if self.head_gate:
+            in_width = -(-in_width // 8) * 8                 # rows stay aligned for vector accesses (checkpoint.stack_rows)
+        self.in_proj = ColumnParallelLinear(hidden_size, in_width, bias=bias, gather_output=False, dtype=dtype,
                                             device=device, tensor_model_parallel_group=tp_group)
         self.o_proj = RowParallelLinear(self.Co, hidden_size, bias=False, input_is_parallel=True, dtype=dtype, device=device,
                                         tensor_model_parallel_group=tp_group)
@@ -120,6 +123,6 @@ class ConvWindowAttention(nn.Module):
         if self.taps:
             ops.short_conv_update(p[..., :C], st, lines, ctx, qlen)
         o = ops.paged_window_attention(q, k_cache, v_cache, meta.block_table, ctx, qlen, self.scale, self.softcap, self.window,
-                                       self.keep_first, p[..., C:] if self.Cg else None, gate_per_head=self.head_gate, chunk=self.chunk,
+                                       self.keep_first, p[..., C:C + self.Cg] if self.Cg else None, gate_per_head=self.head_gate, chunk=self.chunk,
                                        slopes=self.slopes)
         return self.o_proj(o)

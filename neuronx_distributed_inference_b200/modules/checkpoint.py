@@ -195,3 +195,11 @@ def load_sharded(model: nn.Module, full_sd: Dict[str, torch.Tensor], dtype: Opti
             else:
                 dst.copy_(v)
     return sd
+
+
+def stack_rows(*parts, multiple: int = 8):
+    """Projections that read the same input as one matrix, zero rows behind them up to a multiple of ``multiple`` (rows of the product then
+    stay aligned for vector accesses)."""
+    import torch
+    w = torch.cat(parts, 0)
+    return torch.cat([w, w.new_zeros(-w.shape[0] % multiple, *w.shape[1:])], 0)

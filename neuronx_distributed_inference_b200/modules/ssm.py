@@ -221,7 +221,7 @@ class RaggedDecayMixer(nn.Module):
 
 class RaggedMatrixMemoryMixer(nn.Module):
     """Matrix memory with exponential input gates (mLSTM) on ragged rows.  Projection rows are ``[q: heads D | k: heads D | v: heads Dv | out
-    gate: heads Dv | input gate: heads | forget gate: heads]`` in one GEMM (padded with zero rows to a multiple of 8).  Both gates are
+    gate: heads Dv | input gate: heads | forget gate: heads]`` in one GEMM (``checkpoint.stack_rows``: padded to a multiple of 8).  Both gates are
     capped, ``cap tanh(. / cap)`` after their bias; the memory ``S [Dv, D]``, the key sum ``n`` and the running maximum ``m`` of a head follow
     ``m' = max(f + m, i)``, ``S' = e^(f + m - m') S + e^(i - m') v k^T``, ``n'`` likewise with ``k`` alone, and the output is
     ``S' q / (max(|n' . q|, e^-m') + 1e-6)`` with ``q`` scaled by ``D^-1/2``.  Every head is divided by its root mean square, the concatenation
@@ -245,12 +245,6 @@ class RaggedMatrixMemoryMixer(nn.Module):
         self.i_bias = nn.Parameter(torch.zeros(num_heads, **f32), requires_grad=False)
         self.f_bias = nn.Parameter(torch.zeros(num_heads, **f32), requires_grad=False)
         self.norm_weight = nn.Parameter(torch.ones(self.inner, **f32), requires_grad=False)
-
-    @staticmethod
-    def stack(*parts):
-        """The projections in the order of ``in_proj``'s rows, zero rows behind them up to a multiple of 8."""
-        w = torch.cat(parts, 0)
-        return torch.cat([w, w.new_zeros(-w.shape[0] % 8, w.shape[1])], 0)
 
     def _names(self, run):
         run = self.layer_idx if run is None else run

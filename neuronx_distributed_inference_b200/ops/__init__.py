@@ -489,7 +489,7 @@ quantize_blockwise = ref.quantize_blockwise
 # ---- sequence mixers on ragged rows (csrc/seqmix.cu; definitions and conventions in ops/reference.py) ---------------------------
 _MIX_DTYPES = (torch.bfloat16, torch.float32)
 # launch limits of csrc/seqmix.cu (seqmix.h); shapes beyond them run the PyTorch definitions on the same device
-_MIX_MAX_TAPS, _MIX_MAX_VDIM, _MIX_MAX_STATE = 8, 256, 256
+_MIX_MAX_TAPS, _MIX_MAX_VDIM, _MIX_MAX_STATE, _MIX_MAX_ATT_VDIM = 8, 256, 256, 512
 
 
 def _mix_cuda(x) -> bool:
@@ -541,7 +541,7 @@ def conv_qknorm_rope_append(qkv, conv_w, state, slots, ctx_len, q_len, q_norm_w,
 def paged_window_attention(q, k_cache, v_cache, block_table, ctx_len, q_len, scale, softcap, window, keep_first, gate=None, sinks=None,
                            gate_per_head: bool = False, chunk=None, slopes=None, value_dim=None, head_scale=None):
     Dv = v_cache.shape[-1] if value_dim is None else int(value_dim)
-    if _mix_cuda(q) and k_cache.dtype == q.dtype and (gate is None or gate.stride(-1) == 1) and Dv <= _MIX_MAX_VDIM and not (chunk and window):
+    if _mix_cuda(q) and k_cache.dtype == q.dtype and (gate is None or gate.stride(-1) == 1) and Dv <= _MIX_MAX_ATT_VDIM and not (chunk and window):
         stats["paged_window_attention"] += 1
         return _C().paged_window_attention(q.contiguous(), k_cache, v_cache, _i32(block_table), _i32(ctx_len), _i32(q_len), float(scale),
                                            float(softcap or 0.0), int(window or 0), int(keep_first or 0), gate,
@@ -618,7 +618,7 @@ def latent_norm_append(p, offset: int, rank: int, weight, eps: float, cache, blo
 def rope_tail(src, dst, rot_dim: int, cos, sin, interleaved: bool = False):
     """Rotation (rotate-half layout, or pairs (2i, 2i+1) with ``interleaved``) of the last ``rot_dim`` channels of every head of ``src`` into
     the last ``rot_dim`` channels of ``dst``."""
-    rows = src.stride(3) == 1 and src.stride(2) == src.shape[3] and (src.shape[0] == 1 or src.stride(0) == src.shape[1] * src.stride(1))
+    rows = src.stride(3) == 1 and src.stride(2) == src.shape[3] and (src.shape[0] == 1 or src.shape[1] == 1 or src.stride(0) == src.shape[1] * src.stride(1))
     if _mix_cuda(src) and dst.dtype == src.dtype and rows and dst.is_contiguous() and rot_dim % 2 == 0:
         stats["rope_tail"] += 1
         _C().rope_tail(src, dst, int(rot_dim), cos.float().contiguous(), sin.float().contiguous(), bool(interleaved))

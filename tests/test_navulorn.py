@@ -498,9 +498,10 @@ def check_norm_rope_append(dev, dt, tol):
     rn = lambda *s: torch.randn(*s, generator=g)        # noqa: E731
     B, T, page, nblk, eps = 3, 11, 4, 14, 1e-3
     ctx, ql = torch.tensor([0, 5, 40]).int(), torch.tensor([T, 4, 1]).int()
-    for H, G, D, Dv, R in ((4, 2, 10, 6, 8), (3, 1, 10, 7, 6), (2, 2, 16, 16, 0), (4, 2, 64, 128, 64), (2, 1, 12, 8, 2)):
+    for H, G, D, Dv, R in ((4, 2, 10, 6, 8), (3, 1, 10, 7, 6), (2, 2, 16, 16, 0), (4, 2, 64, 128, 64), (2, 1, 12, 8, 2), (5, 1, 24, 16, 16), (6, 3, 128, 64, 96),
+                         (3, 3, 32, 8, 8)):
         C = H * D + G * (D + Dv)
-        p = rn(B, T, C + H).to(dt)
+        p = rn(B, T, -(-(C + H) // 8) * 8).to(dt)
         qw, kw = rn(H * D) * 0.3 + 1, rn(G * D) * 0.3 + 1
         rot = dict(base=77.0, dims=R, scaling=LLAMA31)
         cos, sin = rope_cos_sin(rot, ctx, T, dev) if R else (None, None)
@@ -754,7 +755,8 @@ def test_gpu_other_sizes_and_layouts(tmp_path, dtype, layers, kw):
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("as_prompt", [False, True])
-@pytest.mark.parametrize("latent_rows,D,Dv", [(False, 8, 6), (False, 64, 128), (False, 128, 64), (False, 48, 64), (True, 10, 6), (True, 80, 64), (True, 128, 96)])
+@pytest.mark.parametrize("latent_rows,D,Dv", [(False, 8, 6), (False, 64, 128), (False, 128, 64), (False, 48, 64), (True, 10, 6), (True, 80, 64), (True, 128, 96),
+                                              (True, 410, 400)])
 def test_gpu_loud_keys_near_and_far_and_at_the_windows_edge(dtype, as_prompt, latent_rows, D, Dv):
     for pos, back, window in PLACES:
         got, want, row = loud_key_case("cuda", dtype, pos - back, pos, window, as_prompt=as_prompt, latent_rows=latent_rows, D=D, Dv=Dv)
