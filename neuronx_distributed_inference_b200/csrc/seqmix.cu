@@ -106,12 +106,20 @@ __global__ void __launch_bounds__(256) short_conv_update_kernel(const T* __restr
 }
 
 // ---- convolution + row-wide q / k norm + partial interleaved rotation + paged cache write -------------------------------------
+// query rows past q_len are written as zeros (the output is allocated uninitialised)
+template <typename T>
+__device__ __forceinline__ void zero_query_row(const ConvQkParams& p, int b, int t) {
+  const int Cq = p.n_q * p.D;
+  T* q = (T*)p.q_out + ((long long)b * p.T + t) * Cq;
+  for (int c = threadIdx.x; c < Cq; c += blockDim.x) stf(q + c, 0.f);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) conv_qknorm_rope_append_kernel(ConvQkParams p) {
   extern __shared__ float buf[];      // [Cq + Ck + Cv] convolved row
   __shared__ float red[32];
   const int b = blockIdx.y, t = blockIdx.x;
-  if (t >= p.q_len[b]) return;
+  if (t >= p.q_len[b]) return zero_query_row<T>(p, b, t);
   const int Cq = p.n_q * p.D, Ck = p.n_kv * p.D, Cv = p.n_kv * p.Dv, C = Cq + Ck + Cv, K = p.K;
   const bool has_ctx = p.ctx_len[b] > 0;
   const T* u0 = (const T*)p.p + (long long)b * p.p_sb;
@@ -178,7 +186,7 @@ __global__ void __launch_bounds__(256) conv_qknorm_rope_append_pair_kernel(ConvQ
   extern __shared__ float buf[];      // [Cq + Ck + Cv] convolved row
   __shared__ float red[32];
   const int b = blockIdx.y, t = blockIdx.x;
-  if (t >= p.q_len[b]) return;
+  if (t >= p.q_len[b]) return zero_query_row<T>(p, b, t);
   const int Cq = p.n_q * p.D, Ck = p.n_kv * p.D, Cv = p.n_kv * p.Dv, C = Cq + Ck + Cv, K = p.K;
   const bool has_ctx = p.ctx_len[b] > 0;
   const T* u0 = (const T*)p.p + (long long)b * p.p_sb;
@@ -277,7 +285,7 @@ __global__ void __launch_bounds__(256) qknorm_rope_append_vec_kernel(ConvQkParam
   const int Cq = p.n_q * p.D, Ck = p.n_kv * p.D, Cv = p.n_kv * p.Dv;
   const long long tok = (long long)b * p.T + t;
   T* qo = (T*)p.q_out + tok * Cq;
-  if (t >= p.q_len[b]) return;
+  if (t >= p.q_len[b]) return zero_query_row<T>(p, b, t);
   const T* u = (const T*)p.p + (long long)b * p.p_sb + (long long)t * p.p_st;
   const int pos = p.ctx_len[b] + t;
   long long slot = 0;

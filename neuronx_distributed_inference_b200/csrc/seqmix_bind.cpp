@@ -139,7 +139,7 @@ at::Tensor conv_qknorm_rope_append(const at::Tensor& p, const OptT& conv_w, cons
     a.max_blocks = (int)block_table->size(1);
   }
   c10::cuda::CUDAGuard guard(p.device());
-  auto q = at::zeros({B, T, n_q, D}, p.options());
+  auto q = at::empty({B, T, n_q, D}, p.options());
   a.p = p.data_ptr(); a.p_sb = p.stride(0); a.p_st = p.stride(1);
   a.conv_w = conv_w.has_value() ? conv_w->data_ptr<float>() : nullptr; a.state = K > 1 ? state->data_ptr() : nullptr; a.half = half ? 1 : 0;
   a.lines = lines.data_ptr<int>(); a.ctx_len = ctx.data_ptr<int>(); a.q_len = qlen.data_ptr<int>();
