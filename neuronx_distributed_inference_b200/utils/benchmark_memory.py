@@ -21,7 +21,7 @@ from .benchmark_pairs import VOCAB, build
 from .benchmark_streams import mixers_config as balivik_mixers
 from .benchmark_streams import throughput
 
-BIGRAM = dict(buckets=65521, mul_prev=31, mul_cur=7)
+BIGRAM = dict(buckets=65521, mul_prev=37, mul_cur=11)
 LLAMA31 = dict(factor=8.0, low=1.0, high=4.0, original=8192)
 GATE_CAP = 15.0
 
